@@ -88,6 +88,22 @@ class LukopelConfigC(ctypes.Structure):
                 ("dtype", ctypes.c_int)]
 
 
+class DikopelLayerC(ctypes.Structure):
+    """mirror of ``asd_dikopel_layer_config``"""
+    _fields_ = [(n, ctypes.c_int) for n in (
+        "type", "weights_of", "heads", "dim", "vdim", "a_heads", "a_kv_heads", "a_dim", "a_vdim", "r_heads", "r_kv_heads",
+        "r_dim", "r_vdim", "conv", "ff_kind", "ff", "experts", "top", "expert_ff", "shared_ff", "groups", "keep")] + [
+        (n, ctypes.c_float) for n in ("gate_cap", "scale", "router_scale")]
+
+
+class DikopelConfigC(ctypes.Structure):
+    """mirror of ``asd_dikopel_config``"""
+    _fields_ = [("width", ctypes.c_int), ("vocab", ctypes.c_int), ("n_layers", ctypes.c_int), ("eps", ctypes.c_float),
+                ("embed_scale", ctypes.c_float), ("residual_mult", ctypes.c_float), ("input_taps", ctypes.c_int),
+                ("max_tokens", ctypes.c_int), ("page_size", ctypes.c_int), ("ring", ctypes.c_int),
+                ("dtype", ctypes.c_int)]
+
+
 def library_path() -> str:
     return os.path.join(_HERE, "libasd_b200.so")
 
@@ -181,6 +197,16 @@ def lib() -> ctypes.CDLL:
         "asd_lukopel_forward": (i32, [vp, vp, vp, vp, i32, vp, vp, i32, i32, i32, vp, i32, vp, c.c_longlong, vp, vp]),
         "asd_lukopel_profile_read": (i32, [vp, vp, vp, i32]),
         "asd_lukopel_device_error": (i32, [vp]),
+        "asd_dikopel_create": (vp, [vp, vp]),
+        "asd_dikopel_destroy": (None, [vp]),
+        "asd_dikopel_set_tensor": (i32, [vp, i32, c.c_char_p, vp]),
+        "asd_dikopel_cache_bytes": (sz, [vp, i32]),
+        "asd_dikopel_state_bytes": (sz, [vp, i32]),
+        "asd_dikopel_set_cache": (i32, [vp, vp, i32, vp, i32, i32, vp]),
+        "asd_dikopel_set_option": (i32, [vp, c.c_char_p, i32]),
+        "asd_dikopel_forward": (i32, [vp, vp, vp, vp, i32, vp, vp, i32, i32, i32, vp, i32, vp, c.c_longlong, vp, vp]),
+        "asd_dikopel_profile_read": (i32, [vp, vp, vp, i32]),
+        "asd_dikopel_device_error": (i32, [vp]),
     }
     for name, (res, args) in sigs.items():
         fn = getattr(L, name, None)

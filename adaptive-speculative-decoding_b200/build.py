@@ -28,13 +28,17 @@ COMPONENTS = {
     "rows": ["norm_ops.cu", "moe.cu"],          # row kernels and the expert router that several families share
     "mezilix": ["mezilix_engine.cu", "stream_ops.cu"],
     "rivetar": ["rivetar_engine.cu", "gla.cu", "window_attention.cu"],
-    "mavipel": ["mavipel_engine.cu", "delta_rule.cu", "talking_attention.cu"],
-    "lukopel": ["lukopel_engine.cu", "residual_streams.cu", "mixed_attention.cu", "mixed_attention_tc.cu"],
+    "delta": ["delta_rule.cu"],                 # delta rules and short convolutions
+    "mixattn": ["mixed_attention.cu", "mixed_attention_tc.cu", "sigmoid_attention.cu"],
+    "mavipel": ["mavipel_engine.cu", "talking_attention.cu"],
+    "lukopel": ["lukopel_engine.cu", "residual_streams.cu"],
+    "dikopel": ["dikopel_engine.cu", "mlstm.cu"],
     "qwen": ["engine.cu", "layers.cu", "attention.cu", "attention_tc.cu", "forward_persist.cu"],
     "sampling": ["api.cu", "sampler.cu", "stop_rule.cu"],
 }
 REQUIRES = {"mezilix": ("linear", "blocks", "latent", "rows"), "rivetar": ("linear", "blocks", "latent", "rows"),
-            "mavipel": ("linear", "blocks", "rows"), "lukopel": ("linear", "blocks", "rows"), "qwen": ("linear",)}
+            "mavipel": ("linear", "blocks", "rows", "delta"), "lukopel": ("linear", "blocks", "rows", "mixattn"),
+            "dikopel": ("linear", "blocks", "rows", "delta", "mixattn"), "qwen": ("linear",)}
 
 
 def all_components():

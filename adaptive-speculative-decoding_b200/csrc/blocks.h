@@ -1,5 +1,5 @@
 // Host-side launchers of the sequence-model building blocks that take their sizes and constants as arguments
-// (linear_simt.cu, stream_ops.cu, latent_attention.cu, moe.cu, norm_ops.cu, gla.cu, window_attention.cu).  An engine
+// (linear_simt.cu, stream_ops.cu, latent_attention.cu, moe.cu, norm_ops.cu, gla.cu, window_attention.cu, ...).  An engine
 // (mezilix_engine.cu, rivetar_engine.cu) strings them together;
 // none of them knows a model.  `f32` flags select the element type of a buffer: 0 = bf16, 1 = fp32.  Norms, scores,
 // softmax weights, router probabilities, the residual stream and the carried state are fp32 in both modes.
@@ -146,6 +146,14 @@ struct MoeRouterInput {
     float* logits_out;      // optional [M][E]
     const float* bias = nullptr;   // optional [E], added to the logits
     int renorm = 0;                // 1: the gates are divided by their sum (softmax over the chosen logits alone)
+    // sigmoid = 1: scores s = sigmoid(logit).  The choice goes by s + correction[e] (optional); with groups > 1 the experts
+    // form that many groups of neighbours, a group's score is the sum of its two largest choice scores, and only experts
+    // of the `keep` best groups can be chosen.  gate = s / (sum of the chosen s + 1e-20) * scale.  Needs logits_out.
+    int sigmoid = 0;
+    const float* correction = nullptr;   // [E]
+    int groups = 1, keep = 1;
+    float scale = 1.f;
+    int extra = 0;                 // w has `extra` more rows whose raw logits follow the experts' in logits_out [M][E + extra]
 };
 int launch_moe_route(const float* logits, const MoeRouterInput* in, int M, int E, int top, int* expert_of, float* gate,
                      int* counters, int* group_off, int* sorted_tok, int* slot_of, cudaStream_t stream);
@@ -156,6 +164,10 @@ int launch_moe_route(const float* logits, const MoeRouterInput* in, int M, int E
 // x0[m] = embed[token] * scale, fp32 (x, if given, receives a copy: the stream that the layers go on to change)
 int launch_embed_scaled(const SeqIndex& ix, const void* embed, int wf32, float scale, float* x0, float* x, int D,
                         cudaStream_t stream);
+// x[m] = embed[token] * scale + the sinusoids of the position: sin(p * freq[i]) at coordinate 2 i, cos at 2 i + 1; fp32.
+// freq fp64 [ceil(D / 2)].
+int launch_embed_sinusoid(const SeqIndex& ix, const void* embed, int wf32, float scale, const double* freq, float* x, int D,
+                          cudaStream_t stream);
 // Closes a sublayer and prepares the next one in one pass over a row:
 //   x_out = x_in + (post_w ? y / rms(y) * (1 + post_w) : y) + bias          (each term optional)
 //   hn    = x_out / rms(x_out) * (1 + next_w)   in the engine's element type (if next_w)
@@ -163,6 +175,10 @@ int launch_embed_scaled(const SeqIndex& ix, const void* embed, int wf32, float s
 // plain_w: the weights are taken as they are instead of 1 + w.  groups > 1: the norm before the next sublayer divides
 // each of `groups` equal consecutive parts of the row by its own root mean square.  top > 0: the sum also takes the
 // routed experts' results, gate[m][k] * expert_out[slot_of[m][k]] for k < top in this order (moe.cu).
+// Layers whose sublayers stand side by side: y2 is a second normed branch (y and y2 are then both scaled by y_scale after
+// their norms), ff one more addend, times sigmoid(ff_gate[m * ff_gate_ld]) if given, and everything but x_in is multiplied
+// by mult.  next_b: the norm before the next sublayer is a layer norm (the row's mean is taken off first, next_b added
+// last).  hn_copy: fp32 copy of hn.
 struct RowClose {
     const float* x_in = nullptr;    // [M][D]; with `rows`: row r reads x_in[rows[r]]
     const int* rows = nullptr;
@@ -181,6 +197,15 @@ struct RowClose {
     const int* slot_of = nullptr;       // [M][top]
     const float* gate = nullptr;        // [M][top]
     int top = 0;
+    const float* y2 = nullptr;          // [M][D]
+    const float* post_w2 = nullptr;     // [D]
+    float y_scale = 1.f;
+    const float* ff = nullptr;          // [M][D]
+    const float* ff_gate = nullptr;
+    long long ff_gate_ld = 1;
+    float mult = 1.f;
+    const float* next_b = nullptr;      // [D]
+    float* hn_copy = nullptr;           // [M][D]
 };
 int launch_row_close(const RowClose& c, cudaStream_t stream);
 // x[m] = embed[token] with each of `groups` equal consecutive parts divided by its root mean square, times w; fp32
@@ -268,12 +293,19 @@ int launch_lowrank_channels(const float* a, long long lda, const LowRankChannels
 // the last ring_n new positions of every sequence there and must follow the convolution.
 int launch_short_conv(const SeqIndex& ix, const float* in, long long ld, const float* taps, int n_taps, int C,
                       const float* ring, int ring_n, float* out, cudaStream_t stream);
+// The convolution and the commit in one call (a single launch for steps of one token per sequence).  residual = 0: as
+// above; 1: out[m][c] = in[m][c] + convolution, no activation.  out [M][C] in the engine's element type (of32).
+int launch_carried_conv(const SeqIndex& ix, const int* cu_q, int nseq, int max_qlen, const float* in, long long ld,
+                        const float* taps, int n_taps, int C, float* ring, int ring_n, int residual, void* out, int of32,
+                        cudaStream_t stream);
 int launch_conv_commit(const SeqIndex& ix, const int* cu_q, int nseq, const float* in, long long ld, int C, float* ring,
                        int ring_n, cudaStream_t stream);
-// The vectors a position's recurrence step reads, rv fp32 [M][heads][3 or 5][dk] and sc fp32 [M][heads][4] (layout in
+// The vectors a position's recurrence step reads, rv fp32 [M][heads][3, 2 or 5][dk] and sc fp32 [M][heads][4] (layout in
 // delta_rule.cu).  Gated rule (general = 0): q, k = fp32 rows ld apart holding kv_heads * dk values (head h reads key
 // head h / (heads / kv_heads)), made unit vectors (x / sqrt(sum x^2 + tiny)), q times q_scale; beta = raw rows (ld_beta
-// apart, one per head) that pass a sigmoid; decay fp32 [M][heads * dk].  Generalised rule (general = 1): q = the
+// apart, one per head) that pass a sigmoid; decay fp32 [M][heads * dk], or (general = 2) one per head and position,
+// exp(-exp(head_log_rate[h]) * softplus(rate[m][h] + rate_bias[h])) with rate = raw rows ld_rate apart, and rv then holds
+// only k and q ([2][dk]) while the decay stands in sc.  Generalised rule (general = 1): q = the
 // read-out vectors, k = the keys, rate (raw, ld apart) + rate_bias [heads * dk] pass a sigmoid.
 struct DeltaPrep {
     const float* q = nullptr;
@@ -284,6 +316,8 @@ struct DeltaPrep {
     long long ld_beta = 0;
     const float* rate = nullptr;
     const float* rate_bias = nullptr;
+    const float* head_log_rate = nullptr;
+    long long ld_rate = 0;
     float* rv = nullptr;
     float* sc = nullptr;
     int heads = 0, kv_heads = 0, dk = 0, general = 0;
@@ -297,12 +331,13 @@ int launch_delta_recurrence(const SeqIndex& ix, const int* cu_q, const int* seq_
                             const float* sc, int general, const float* v, long long ldv, int heads, int dk, int dv,
                             float* state, int ring, float* out, cudaStream_t stream);
 // y[m][h][:] = o[m][h][:] / rms(o[m][h][:]) * w * gate[m][h][:] * scale, y = rows ldy apart in the engine's element
-// type.  w: [dv] shared by the heads or [heads * dv]; gate: fp32 rows ldg apart, taken as they are or through a sigmoid.
+// type.  w: [dv] shared by the heads or [heads * dv]; gate: fp32 rows ldg apart, taken as they are (gate_act 0), through a
+// sigmoid (1) or a silu (2).
 struct HeadNormGate {
     const float* gate = nullptr;
     long long ldg = 0;
     const float* w = nullptr;
-    int w_per_head = 0, gate_sigmoid = 0;
+    int w_per_head = 0, gate_act = 0;
     float eps = 0.f, scale = 1.f;
 };
 int launch_head_norm_gate(const float* o, const HeadNormGate& p, void* y, int of32, long long ldy, int M, int heads, int dv,
@@ -368,6 +403,9 @@ struct MixDims {
     int heads, kv_heads, dk, dv;
     int chunk;          // 0: position i sees every j <= i; else only those with j / chunk == i / chunk
     float scale;
+    // 1: the weight of a visible key is sigmoid(score + head_bias[head]), not normalised over the keys (no head mix then)
+    int sigmoid = 0;
+    const float* head_bias = nullptr;   // fp32 [heads], optional
 };
 // What the projections pass before the attention.  qkv fp32 rows (ld floats apart) = [heads * dk | kv_heads * dk |
 // kv_heads * dv].  Adds the biases (same layout, optional); RMS-norms queries and keys either head by head (weights [dk],
@@ -409,6 +447,36 @@ int launch_mix_attention(const SeqIndex& ix, const int* cu_q, const int* seq_slo
                          const float* q, long long ldq, const MixDims& d, const float* dist_bias, int far,
                          const float* talk, const float* gate, long long ldg, const PagedRows& cache, void* out, int of32,
                          long long ldo, const MixWork& ws, cudaStream_t stream);
+
+// ---------------------------------------------------------------------------------------------- mlstm.cu
+// Matrix memory with exponential gates (mLSTM): per head a state S [dk][dv], a normaliser n [dk] and a running maximum M,
+//   M' = max(f + M, i);  S = exp(f + M - M') S + exp(i - M') k v^T;  n likewise with k alone;
+//   o = S^T q / (max(|n . q|, exp(-M')) + 1e-6),
+// with logarithmic gates i = cap tanh(zi / cap) and f = log_sigmoid(cap tanh(zf / cap)).
+struct MlstmDims {
+    int heads, dk, dv;
+    float cap;
+    float q_scale;      // scale of the queries
+};
+// What a recurrence step reads: fp32 rows ld floats apart, q and k (heads * dk used), v (heads * dv), and one raw gate value
+// per head, to which the biases are added.
+struct MlstmInput {
+    const float* q = nullptr;
+    const float* k = nullptr;
+    const float* v = nullptr;
+    const float* zi = nullptr;
+    const float* zf = nullptr;
+    long long ld = 0;
+    const float* bias_i = nullptr;   // [heads]
+    const float* bias_f = nullptr;
+};
+// floats of state per sequence and ring entry: heads * (dk * dv + ceil(dv / 32) * (dk + 1))
+size_t mlstm_state_elems(const MlstmDims& d);
+// state fp32 [slots][ring][ S [heads][dk][dv] | [heads][ceil(dv / 32)] x (n [dk], M) ]; entry position % ring holds the state after that
+// position.  A sequence whose first new position is 0 starts from zero, any other from entry (position - 1) % ring; the
+// last `ring` new positions of a sequence store theirs.  out fp32 [M][heads * dv].
+int launch_mlstm_recurrence(const SeqIndex& ix, const int* cu_q, const int* seq_slot, int nseq, const MlstmInput& in,
+                            const MlstmDims& d, float* state, int ring, float* out, cudaStream_t stream);
 
 int preload_blocks();
 

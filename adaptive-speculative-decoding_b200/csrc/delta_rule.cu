@@ -11,7 +11,8 @@
 // of the updated state is expanded, so that one pass over the old state serves the correction and the result); five
 // vectors per position (w, n, w * r, k, a * n).  Gated rule, in the order it is written: S[r] <- g[r] S[r], then
 // A = sum_r S[r] k[r] and B = sum_r S[r] q[r] in the same pass, u = beta (v - A), S[r] <- S[r] + k[r] u (k still in
-// registers: nothing is read after the exchange), o = B + u (k . q); three vectors per position (g, k, q).  delta_prep_kernel forms these vectors; delta_recurrence_kernel holds a CTA's 32 value columns of the state
+// registers: nothing is read after the exchange), o = B + u (k . q); three vectors per position (g, k, q), or two (k, q)
+// where the decay is one number per head and position.  delta_prep_kernel forms these vectors; delta_recurrence_kernel holds a CTA's 32 value columns of the state
 // in registers, the key rows cut into slices over its warps, for the whole run of new positions.  The arithmetic per
 // position is the same whatever the chunking or the batch.  State: fp32 [slot][ring][head][dk][dv], entry p % ring =
 // the state after position p.
@@ -88,33 +89,45 @@ __global__ void __launch_bounds__(LC_CH) lowrank_channels_kernel(const float* a,
 // ------------------------------------------------------------------------------------------ short causal convolution
 // out[m][c] = silu( sum_j taps[c][j] * in[position - (n - 1 - j)][c] ): inputs of this forward come from the rows above
 // (a sequence's tokens are consecutive rows), earlier ones from the ring of carried inputs, zeros before position 0.
+// RESID: out = in + convolution, no activation, in the engine's element type.  SINGLE (one token per sequence): the thread
+// that has read a channel's carried inputs stores its new one, which saves the commit launch; the entry it overwrites is
+// either the oldest input, read by this very thread, or older than any that is read.
+template <bool RESID, bool SINGLE>
 __global__ void short_conv_kernel(SeqIndex ix, const float* in, long long ld, const float* taps, int n, int C,
-                                  const float* ring, int ring_n, float* out) {
+                                  const float* ring_in, float* ring, int ring_n, void* out, int of32) {
     const int m = blockIdx.x;
     const int pos = ix.positions[m], slot = ix.token_slot[m];
     // how many rows above belong to the same sequence's preceding positions (at most n - 1 are needed)
     int above = 0;
-    while (above < n - 1 && m - above - 1 >= 0 && ix.token_slot[m - above - 1] == slot &&
-           ix.positions[m - above - 1] == pos - above - 1)
-        ++above;
+    if (!SINGLE)
+        while (above < n - 1 && m - above - 1 >= 0 && ix.token_slot[m - above - 1] == slot &&
+               ix.positions[m - above - 1] == pos - above - 1)
+            ++above;
     // four channels per thread, blockDim apart, their loads independent of one another
     const int cb = blockIdx.y * blockDim.x * 4 + threadIdx.x;
-    float acc[4] = {0.f, 0.f, 0.f, 0.f};
+    float acc[4] = {0.f, 0.f, 0.f, 0.f}, cur[4] = {0.f, 0.f, 0.f, 0.f};
     for (int j = 0; j < n; ++j) {
         const int back = n - 1 - j;       // taps' last column weighs the current position
         const int p = pos - back;
         if (p < 0) continue;
-        const float* src = back <= above ? in + (long long)(m - back) * ld : ring + ((long long)slot * ring_n + p % ring_n) * C;
+        const float* src = back <= above ? in + (long long)(m - back) * ld : ring_in + ((long long)slot * ring_n + p % ring_n) * C;
 #pragma unroll
         for (int u = 0; u < 4; ++u) {
             const int c = cb + u * blockDim.x;
-            if (c < C) acc[u] = fmaf(__ldg(taps + (long long)c * n + j), __ldg(src + c), acc[u]);
+            if (c < C) {
+                const float v = SINGLE && back > 0 ? src[c] : __ldg(src + c);
+                if (back == 0) cur[u] = v;
+                acc[u] = fmaf(__ldg(taps + (long long)c * n + j), v, acc[u]);
+            }
         }
     }
 #pragma unroll
     for (int u = 0; u < 4; ++u) {
         const int c = cb + u * blockDim.x;
-        if (c < C) out[(long long)m * C + c] = acc[u] / (1.f + expf(-acc[u]));
+        if (c < C) {
+            stx(out, (long long)m * C + c, of32, RESID ? cur[u] + acc[u] : acc[u] / (1.f + expf(-acc[u])));
+            if (SINGLE) ring[((long long)slot * ring_n + pos % ring_n) * C + c] = cur[u];
+        }
     }
 }
 
@@ -132,18 +145,20 @@ __global__ void conv_commit_kernel(SeqIndex ix, const int* cu_q, const float* in
 }
 
 // ------------------------------------------------------------------------------------------ a position's vectors
-// one warp per (token, head): rv[m][h][vec][dk] with vec = g, k, q (gated) or w, n, w * r, k, a * n (generalised) and
-// sc[m][h][4] = beta, -, k . q, - (gated) or -, -, (a * n) . r, k . r (generalised)
+__host__ __device__ inline int delta_vectors(int general) { return general == 0 ? 3 : (general == 1 ? 5 : 2); }
+
+// one warp per (token, head): rv[m][h][vec][dk] with vec = g, k, q (gated), k, q (gated, decay per head) or w, n, w * r,
+// k, a * n (generalised) and sc[m][h][4] = beta, -, k . q, - or beta, g, k . q, - or -, -, (a * n) . r, k . r
 __global__ void delta_prep_kernel(DeltaPrep p, int M) {
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const long long idx = (long long)blockIdx.x * (blockDim.x >> 5) + warp;
     if (idx >= (long long)M * p.heads) return;
     const int m = (int)(idx / p.heads), h = (int)(idx - (long long)m * p.heads);
-    const int dk = p.dk, nv = p.general ? 5 : 3;
+    const int dk = p.dk, nv = delta_vectors(p.general);
     const int kvh = h / (p.heads / p.kv_heads);
     const float* q = p.q + (long long)m * p.ld + (long long)kvh * dk;
     const float* k = p.k + (long long)m * p.ld + (long long)kvh * dk;
-    const float* d = p.decay + ((long long)m * p.heads + h) * dk;
+    const float* d = p.decay ? p.decay + ((long long)m * p.heads + h) * dk : nullptr;
     float* rv = p.rv + ((long long)m * p.heads + h) * nv * dk;
     float kk = 0.f, qq = 0.f;
     for (int i = lane; i < dk; i += 32) {
@@ -154,20 +169,28 @@ __global__ void delta_prep_kernel(DeltaPrep p, int M) {
     qq = warp_sum(qq);
     const float kn = 1.f / sqrtf(kk + p.tiny);
     float s1 = 0.f, s2 = 0.f;
-    if (!p.general) {
+    if (p.general != 1) {
         const float qn = p.q_scale / sqrtf(qq + p.tiny);
         for (int i = lane; i < dk; i += 32) {
-            const float kv = k[i] * kn, qv = q[i] * qn, dv = d[i];
-            rv[i] = dv;
-            rv[dk + i] = kv;
-            rv[2 * dk + i] = qv;
+            const float kv = k[i] * kn, qv = q[i] * qn;
+            if (p.general == 0) {
+                rv[i] = d[i];
+                rv[dk + i] = kv;
+                rv[2 * dk + i] = qv;
+            } else {
+                rv[i] = kv;
+                rv[dk + i] = qv;
+            }
             s1 = fmaf(kv, qv, s1);
         }
         s1 = warp_sum(s1);
         if (lane == 0) {
             const float beta = sigmoid_f(p.beta[(long long)m * p.ld_beta + h]);
+            float g = beta;
+            if (p.general == 2)      // 1 + expm1: a decay just below 1 is rounded once
+                g = 1.f + expm1f(-expf(p.head_log_rate[h]) * softplus_f(p.rate[(long long)m * p.ld_rate + h] + p.rate_bias[h]));
             float* sc = p.sc + ((long long)m * p.heads + h) * 4;
-            sc[0] = beta, sc[1] = beta, sc[2] = s1, sc[3] = s1;
+            sc[0] = beta, sc[1] = g, sc[2] = s1, sc[3] = s1;
         }
     } else {
         const float* a = p.rate + (long long)m * p.ld + (long long)h * dk;
@@ -204,7 +227,7 @@ __device__ __forceinline__ void cp_async16(float* dst, const float* src) {
 }
 
 // ROWS state rows per thread; warps = slices of ROWS key rows (rows beyond dk are staged as zeros and keep a zero
-// state).  NV = 3: the gated rule; NV = 5: the generalised rule.  CH positions are staged per chunk by
+// state).  NV = 3: the gated rule; 2: the gated rule with one decay per head; 5: the generalised rule.  CH positions are staged per chunk by
 // cp.async, one chunk ahead of the arithmetic.
 template <int ROWS, int NV, int MAXT>
 __global__ void __launch_bounds__(MAXT, 1) delta_recurrence_kernel(SeqIndex ix, const int* cu_q, const int* seq_slot,
@@ -288,14 +311,16 @@ __global__ void __launch_bounds__(MAXT, 1) delta_recurrence_kernel(SeqIndex ix, 
             const float4* d4 = reinterpret_cast<const float4*>(vt);
             float* rp = red + (size_t)par * RS * 64;
             float o_t;
-            if constexpr (NV == 3) {
-                const float4* k4 = reinterpret_cast<const float4*>(vt + dkp);
-                const float4* q4 = reinterpret_cast<const float4*>(vt + 2 * dkp);
+            if constexpr (NV <= 3) {
+                const float4* k4 = reinterpret_cast<const float4*>(vt + (NV - 2) * dkp);
+                const float4* q4 = reinterpret_cast<const float4*>(vt + (NV - 1) * dkp);
+                const float g = ss[t * 4 + 1];
                 float kr[ROWS];
                 float a0 = 0.f, a1 = 0.f, b0 = 0.f, b1 = 0.f;
 #pragma unroll
                 for (int r = 0; r < ROWS; r += 4) {
-                    const float4 dd = d4[r >> 2], kk = k4[r >> 2], qq = q4[r >> 2];
+                    const float4 kk = k4[r >> 2], qq = q4[r >> 2];
+                    const float4 dd = NV == 2 ? make_float4(g, g, g, g) : d4[r >> 2];
                     kr[r] = kk.x, kr[r + 1] = kk.y, kr[r + 2] = kk.z, kr[r + 3] = kk.w;
                     S[r] *= dd.x, S[r + 1] *= dd.y, S[r + 2] *= dd.z, S[r + 3] *= dd.w;
                     a0 = fmaf(S[r], kk.x, a0);
@@ -453,14 +478,16 @@ __global__ void __launch_bounds__(512, 1) delta_recurrence_cols_kernel(SeqIndex 
         for (int t = 0; t < nt; ++t) {
             const float4* d4 = reinterpret_cast<const float4*>(vec + t * NV * DKP + part * PS);
             float o_t;
-            if constexpr (NV == 3) {
-                const float4* k4 = d4 + DKP / 4;
-                const float4* q4 = d4 + 2 * (DKP / 4);
+            if constexpr (NV <= 3) {
+                const float4* k4 = d4 + (NV - 2) * (DKP / 4);
+                const float4* q4 = d4 + (NV - 1) * (DKP / 4);
+                const float g = ss[t * 4 + 1];
                 float kr[ROWS];
                 float a0 = 0.f, a1 = 0.f, b0 = 0.f, b1 = 0.f;
 #pragma unroll
                 for (int r = 0; r < ROWS; r += 4) {
-                    const float4 dd = d4[r >> 2], kk = k4[r >> 2], qq = q4[r >> 2];
+                    const float4 kk = k4[r >> 2], qq = q4[r >> 2];
+                    const float4 dd = NV == 2 ? make_float4(g, g, g, g) : d4[r >> 2];
                     kr[r] = kk.x, kr[r + 1] = kk.y, kr[r + 2] = kk.z, kr[r + 3] = kk.w;
                     S[r] *= dd.x, S[r + 1] *= dd.y, S[r + 2] *= dd.z, S[r + 3] *= dd.w;
                     a0 = fmaf(S[r], kk.x, a0);
@@ -546,7 +573,8 @@ __global__ void head_norm_gate_kernel(const float* o, HeadNormGate p, void* y, i
     ss = warp_sum(ss);
     const float r = p.scale / sqrtf(ss / (float)dv + p.eps);
     for (int i = lane; i < dv; i += 32) {
-        const float gv = p.gate_sigmoid ? sigmoid_f(g[i]) : g[i];
+        float gv = g[i];
+        if (p.gate_act) gv = (p.gate_act == 2 ? gv : 1.f) * sigmoid_f(gv);
         stx(y, m * ldy + (long long)h * dv + i, of32, src[i] * r * w[i] * gv);
     }
 }
@@ -571,18 +599,48 @@ int launch_lowrank_channels(const float* a, long long lda, const LowRankChannels
     return 0;
 }
 
+static int short_conv_check(int n_taps, const float* ring, int ring_n) {
+    if (n_taps <= 0 || (n_taps > 1 && (!ring || ring_n < n_taps - 1)))
+        return set_error("short_conv: %d taps need a ring of at least %d carried inputs", n_taps, n_taps - 1);
+    return 0;
+}
+
 int launch_short_conv(const SeqIndex& ix, const float* in, long long ld, const float* taps, int n_taps, int C,
                       const float* ring, int ring_n, float* out, cudaStream_t stream) {
     if (ix.M <= 0 || C <= 0) return 0;
-    if (n_taps <= 0 || (n_taps > 1 && (!ring || ring_n < n_taps - 1)))
-        return set_error("short_conv: %d taps need a ring of at least %d carried inputs", n_taps, n_taps - 1);
+    if (short_conv_check(n_taps, ring, ring_n)) return -1;
     const int threads = C >= 1024 ? 256 : 128;
     dim3 grid(ix.M, (C + 4 * threads - 1) / (4 * threads));
     if (grid.y > 65535) return set_error("short_conv: too many channels");
-    short_conv_kernel<<<grid, threads, 0, stream>>>(ix, in, ld, taps, n_taps, C, ring, ring_n > 0 ? ring_n : 1, out);
+    short_conv_kernel<false, false><<<grid, threads, 0, stream>>>(ix, in, ld, taps, n_taps, C, ring, nullptr,
+                                                                  ring_n > 0 ? ring_n : 1, out, 1);
     count_launch(1);
     ASD_CUDA(cudaGetLastError());
     return 0;
+}
+
+int launch_carried_conv(const SeqIndex& ix, const int* cu_q, int nseq, int max_qlen, const float* in, long long ld,
+                        const float* taps, int n_taps, int C, float* ring, int ring_n, int residual, void* out, int of32,
+                        cudaStream_t stream) {
+    if (ix.M <= 0 || C <= 0) return 0;
+    if (short_conv_check(n_taps, ring, ring_n)) return -1;
+    const bool single = max_qlen == 1 && ring_n > 0 && n_taps > 1;
+    const int threads = C >= 1024 ? 256 : 128;
+    dim3 grid(ix.M, (C + 4 * threads - 1) / (4 * threads));
+    if (grid.y > 65535) return set_error("short_conv: too many channels");
+    const int rn = ring_n > 0 ? ring_n : 1;
+    if (residual && single)
+        short_conv_kernel<true, true><<<grid, threads, 0, stream>>>(ix, in, ld, taps, n_taps, C, ring, ring, rn, out, of32);
+    else if (residual)
+        short_conv_kernel<true, false><<<grid, threads, 0, stream>>>(ix, in, ld, taps, n_taps, C, ring, nullptr, rn, out, of32);
+    else if (single)
+        short_conv_kernel<false, true><<<grid, threads, 0, stream>>>(ix, in, ld, taps, n_taps, C, ring, ring, rn, out, of32);
+    else
+        short_conv_kernel<false, false><<<grid, threads, 0, stream>>>(ix, in, ld, taps, n_taps, C, ring, nullptr, rn, out, of32);
+    count_launch(1);
+    ASD_CUDA(cudaGetLastError());
+    if (single || ring_n <= 0) return 0;
+    return launch_conv_commit(ix, cu_q, nseq, in, ld, C, ring, ring_n, stream);
 }
 
 int launch_conv_commit(const SeqIndex& ix, const int* cu_q, int nseq, const float* in, long long ld, int C, float* ring,
@@ -599,7 +657,9 @@ int launch_delta_prep(const DeltaPrep& p, int M, cudaStream_t stream) {
     if (M <= 0) return 0;
     if (p.heads <= 0 || p.kv_heads <= 0 || p.heads % p.kv_heads || p.dk <= 0)
         return set_error("delta_prep: %d heads over %d key heads of size %d", p.heads, p.kv_heads, p.dk);
-    if (p.general ? (!p.rate || !p.rate_bias) : !p.beta) return set_error("delta_prep: missing inputs");
+    if ((p.general ? (!p.rate || !p.rate_bias) : !p.decay) || (p.general != 1 && !p.beta) ||
+        (p.general == 1 && !p.decay) || (p.general == 2 && !p.head_log_rate))
+        return set_error("delta_prep: missing inputs");
     const long long pairs = (long long)M * p.heads;
     delta_prep_kernel<<<(unsigned)((pairs + 7) / 8), 256, 0, stream>>>(p, M);
     count_launch(1);
@@ -617,7 +677,7 @@ int launch_delta_recurrence(const SeqIndex& ix, const int* cu_q, const int* seq_
     // steps of single tokens: the state is read and written once per position and the shuffle form keeps more loads in
     // flight; prompts and portions: the slices over warps read every staged vector once per warp as a broadcast
     if (ix.M <= 2 * nseq && dk <= 128 && ((dv + 32 / parts - 1) / (32 / parts)) * 32 <= 512) {   // row blocks closed by shuffles: no barrier per position
-        const int nvv = general ? 5 : 3, dkp = 36 * parts;
+        const int nvv = delta_vectors(general), dkp = 36 * parts;
         const int cpw = 32 / parts, warps = (dv + cpw - 1) / cpw, dvp = warps * cpw;
         int ch = 16;   // positions per staged chunk; steps of few tokens per sequence stage (and clear) no more than they use
         while (ch > 1 && (long long)(ch / 2) * nseq >= ix.M) ch >>= 1;
@@ -637,8 +697,10 @@ int launch_delta_recurrence(const SeqIndex& ix, const int* cu_q, const int* seq_
     if (parts == 1) ASD_DC_CASE(1, NVV)          \
     else if (parts == 2) ASD_DC_CASE(2, NVV)     \
     else ASD_DC_CASE(4, NVV)
-        if (general) {
+        if (general == 1) {
             ASD_DC_PARTS(5)
+        } else if (general == 2) {
+            ASD_DC_PARTS(2)
         } else {
             ASD_DC_PARTS(3)
         }
@@ -651,7 +713,7 @@ int launch_delta_recurrence(const SeqIndex& ix, const int* cu_q, const int* seq_
     int rows = 4;
     while (rows < 32 && rows * 4 < dk) rows *= 2;     // four warps up to key size 128, then more
     const int RS = (dk + rows - 1) / rows;
-    const int dkp = RS * rows, nv = general ? 5 : 3;
+    const int dkp = RS * rows, nv = delta_vectors(general);
     int ch = 16;   // positions per staged chunk: as many as two buffers of a head's vectors leave room for
     while (ch > 1 && (long long)(ch / 2) * nseq >= ix.M) ch >>= 1;
     auto need = [&](int c) { return (size_t)(2 * (c * nv * dkp + c * 36) + 2 * RS * 64) * sizeof(float); };
@@ -673,8 +735,10 @@ int launch_delta_recurrence(const SeqIndex& ix, const int* cu_q, const int* seq_
     else if (rows == 8) ASD_DR_CASE(8, NVV, 256)     \
     else if (rows == 16) ASD_DR_CASE(16, NVV, 256)   \
     else ASD_DR_CASE(32, NVV, 256)
-    if (general) {
+    if (general == 1) {
         ASD_DR_ROWS(5)
+    } else if (general == 2) {
+        ASD_DR_ROWS(2)
     } else {
         ASD_DR_ROWS(3)
     }

@@ -156,7 +156,7 @@ static int mix_channel_delta(MvEngine* e, const MvLayer& ly, const MvRun& run, i
     dp.q_scale = 1.f / sqrtf((float)c.dim);
     dp.beta = e->proj + 2 * nk + nv, dp.ld_beta = ly.ld_in;   // the raw betas stay in the projection's rows
     HeadNormGate ng;
-    ng.gate = e->gatev, ng.ldg = nv, ng.w = ly.f("out_norm"), ng.w_per_head = 0, ng.gate_sigmoid = 0, ng.eps = e->c.eps;
+    ng.gate = e->gatev, ng.ldg = nv, ng.w = ly.f("out_norm"), ng.w_per_head = 0, ng.gate_act = 0, ng.eps = e->c.eps;
     return delta_core(e, b, dp, e->conv + 2 * nk, ly.conv_ch, c.vdim, e->state + run.state_off, ng, ly.mix_w, 0, s);
 }
 
@@ -194,7 +194,7 @@ static int mix_parallel(MvEngine* e, const MvLayer& ly, const MvRun& run, int li
     dp.q = r, dp.k = r + nr, dp.ld = ly.ld_in, dp.decay = e->decay, dp.rate = r + 4 * nr, dp.rate_bias = ly.f("rate_bias");
     dp.rv = e->rv, dp.sc = e->sc, dp.heads = c.r_heads, dp.kv_heads = c.r_heads, dp.dk = c.r_dim, dp.general = 1;
     HeadNormGate ng;
-    ng.gate = r + 3 * nr, ng.ldg = ly.ld_in, ng.w = ly.f("out_norm"), ng.w_per_head = 1, ng.gate_sigmoid = 1;
+    ng.gate = r + 3 * nr, ng.ldg = ly.ld_in, ng.w = ly.f("out_norm"), ng.w_per_head = 1, ng.gate_act = 1;
     ng.eps = e->c.eps, ng.scale = c.right_scale;
     return delta_core(e, b, dp, r + 2 * nr, ly.ld_in, c.r_dim, e->state + run.state_off, ng, ly.mix_w,
                       c.a_heads * c.a_vdim, s);

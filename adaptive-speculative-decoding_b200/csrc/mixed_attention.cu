@@ -9,6 +9,7 @@
 // Because the weights are normalised with the final statistics, the key shares' partial results simply add (merge kernel,
 // fixed order).  Scores, weights and sums are fp32; keys and values come from the paged cache in its element type.
 // Without mixing (talk == nullptr) the same two passes run with one key/value group per CTA.
+// Sigmoid weights (MixDims.sigmoid) need no statistics: w_g = sigmoid(score + head_bias[g]) in one pass over the keys.
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
 #include <math.h>
@@ -144,7 +145,7 @@ __global__ void __launch_bounds__(NT) mix_attn_kernel(MixArgs a) {
     if (APPLY) {
         if (a.talk)
             for (int i = tid; i < H * H; i += NT) talk_s[i] = a.talk[i];
-        for (int row = tid; row < rows; row += NT) {   // final statistics: the key shares' maxima and sums merged
+        for (int row = tid; row < rows && !a.d.sigmoid; row += NT) {   // final statistics: the key shares' maxima and sums merged
             const int h = hbeg + row / QT, i = row % QT;
             float mm = -INFINITY, ll = 0.f;
             if (i < nq) {
@@ -252,6 +253,12 @@ __global__ void __launch_bounds__(NT) mix_attn_kernel(MixArgs a) {
                             lrun[rc][x] = lrun[rc][x] * keep + sum;
                             mrun[rc][x] = mnew;
                         }
+                    } else if (row_ok && a.d.sigmoid) {
+                        const float hb = a.d.head_bias ? a.d.head_bias[h] : 0.f;
+#pragma unroll
+                        for (int y = 0; y < 4; ++y)
+                            Pm[(size_t)(lrow0 + rg) * PS + tx + 16 * y] =
+                                s[y] > -INFINITY ? 1.f / (1.f + expf(-(s[y] + hb))) : 0.f;
                     } else if (row_ok) {
                         const int lrow = lrow0 + rg;
                         const float mm = Mr[lrow], il = Lr[lrow];
@@ -809,6 +816,7 @@ int mix_attention_check(const MixDims& d, int talk) {
     if (d.dv > 256) return set_error("mixed attention: value size %d above 256", d.dv);
     if (d.dk > 512) return set_error("mixed attention: key size %d above 512", d.dk);
     if (d.heads / d.kv_heads > MAX_ROWS) return set_error("mixed attention: more than %d query heads per key head", MAX_ROWS);
+    if (talk && d.sigmoid) return set_error("mixed attention: sigmoid weights are not mixed across heads");
     if (talk && d.heads > MAX_ROWS) return set_error("mixed attention: more than %d heads with mixed weights", MAX_ROWS);
     return 0;
 }
@@ -829,7 +837,8 @@ int launch_mix_attention(const SeqIndex& ix, const int* cu_q, const int* seq_slo
     a.vec = (d.dk % 4 == 0 && d.dv % 4 == 0) ? 1 : 0;
     // steps of few tokens; prompts of a bf16 engine on the tensor cores; else (and for sizes those refuse) the CUDA cores
     if (max_qlen <= 4 && ws.mode != 1) {
-        const int rc = launch_mix_attention_decode(a, nseq, max_kv_len, ws, stream);
+        const int rc = d.sigmoid ? launch_sigmoid_attention_decode(a, max_kv_len, ws, stream)
+                                 : launch_mix_attention_decode(a, nseq, max_kv_len, ws, stream);
         if (rc <= 0) return rc;
     }
     if (!cache.f32 && ws.mode != 1) {
@@ -859,28 +868,29 @@ int launch_mix_attention(const SeqIndex& ix, const int* cu_q, const int* seq_slo
     int shares = 1;
     const long long base = (long long)tiles * nseq * ngroups;
     const int key_tiles = (max_kv_len + KT - 1) / KT;
-    if (base < 148 && ws.stats && ws.part) {
+    const long long stat_rows = d.sigmoid ? 0 : (long long)2 * ix.M * H;     // workspace floats per share
+    if (base < 148 && (ws.stats || d.sigmoid) && ws.part) {
         shares = (int)std::min<long long>((296 + base - 1) / base, (long long)std::max(1, key_tiles / 2));
         shares = std::min(shares, 32);
         while (shares > 1 && ((long long)shares * ix.M * H * d.dv > ws.part_elems ||
-                              (long long)2 * shares * ix.M * H > ws.stats_elems))
+                              shares * stat_rows > ws.stats_elems))
             --shares;
     }
-    if ((long long)2 * shares * ix.M * H > ws.stats_elems || !ws.stats)
+    if (!d.sigmoid && (shares * stat_rows > ws.stats_elems || !ws.stats))
         return set_error("mixed attention: statistics workspace too small");
     a.shares = shares;
     const size_t smem_stats = (size_t)mix_layout(rep * QT, dkp, dvp, H, false, false).total * sizeof(float);
     const dim3 gs(tiles, nseq, shares * G), ga(tiles, nseq, shares * ngroups);
     const int cb = dvp <= 64 ? 1 : (dvp <= 128 ? 2 : 4);
-    int rc;
+    int rc = 0;
     if (cache.f32) {
-        rc = launch_one<float, false, 1>(a, gs, smem_stats, stream);
+        if (!d.sigmoid) rc = launch_one<float, false, 1>(a, gs, smem_stats, stream);
         if (!rc)
             rc = cb == 1 ? launch_one<float, true, 1>(a, ga, smem_apply, stream)
                          : (cb == 2 ? launch_one<float, true, 2>(a, ga, smem_apply, stream)
                                     : launch_one<float, true, 4>(a, ga, smem_apply, stream));
     } else {
-        rc = launch_one<__nv_bfloat16, false, 1>(a, gs, smem_stats, stream);
+        if (!d.sigmoid) rc = launch_one<__nv_bfloat16, false, 1>(a, gs, smem_stats, stream);
         if (!rc)
             rc = cb == 1 ? launch_one<__nv_bfloat16, true, 1>(a, ga, smem_apply, stream)
                          : (cb == 2 ? launch_one<__nv_bfloat16, true, 2>(a, ga, smem_apply, stream)

@@ -74,10 +74,13 @@ __device__ __forceinline__ void stage_rows(const bf16* pool, const long long* ro
     }
 }
 
-// ONE (second pass without a head mix, all keys in one share): no first pass at all; the running maximum rescales the
-// sums tile by tile and the division by the softmax sum comes last.
-template <int KT, int NDV, bool APPLY, bool TALK, bool ONE>
+// MODE of the second pass.  TWO_PASS: weights normalised with the first pass's statistics.  ONLINE (no head mix, all keys in
+// one share): no first pass at all; the running maximum rescales the sums tile by tile and the division by the softmax sum
+// comes last.  SIGMOID: the weights are sigmoids and need no statistics.
+enum { TWO_PASS = 0, ONLINE = 1, SIGMOID = 2 };
+template <int KT, int NDV, bool APPLY, bool TALK, int MODE>
 __global__ void __launch_bounds__(NT) mix_tc_kernel(MixArgs a) {
+    constexpr bool ONE = MODE == ONLINE;
     extern __shared__ __align__(16) unsigned char smraw[];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
     const int H = a.d.heads, G = a.d.kv_heads, rep = H / G, dk = a.d.dk, dv = a.d.dv, QT = a.QT, chunk = a.d.chunk;
@@ -122,7 +125,7 @@ __global__ void __launch_bounds__(NT) mix_tc_kernel(MixArgs a) {
         Qh[(size_t)row * DS + d] = hi;
         Ql[(size_t)row * DS + d] = __float2bfloat16(v - __bfloat162float(hi));
     }
-    if (APPLY && !ONE) {
+    if (APPLY && MODE == TWO_PASS) {
         if (TALK)
             for (int i = tid; i < H * H; i += NT) talk_s[i] = a.talk[i];
         for (int row = tid; row < rows; row += NT) {   // final statistics: the key shares' maxima and sums merged
@@ -163,7 +166,7 @@ __global__ void __launch_bounds__(NT) mix_tc_kernel(MixArgs a) {
     const bool active = rb < rows;
     int hx[2], ix_[2], posx[2], lox[2];
     bool okx[2];
-    float Mx[2] = {0.f, 0.f}, iLx[2] = {0.f, 0.f};
+    float Mx[2] = {0.f, 0.f}, iLx[2] = {0.f, 0.f}, hbx[2] = {0.f, 0.f};
 #pragma unroll
     for (int x = 0; x < 2; ++x) {
         const int r = active ? rb + g + 8 * x : 0;
@@ -171,7 +174,8 @@ __global__ void __launch_bounds__(NT) mix_tc_kernel(MixArgs a) {
         posx[x] = p0 + ix_[x];
         lox[x] = chunk > 0 ? (posx[x] / chunk) * chunk : 0;
         okx[x] = active && ix_[x] < nq;
-        if (APPLY && !ONE && active) Mx[x] = Mr[r], iLx[x] = Lr[r];
+        if (APPLY && MODE == TWO_PASS && active) Mx[x] = Mr[r], iLx[x] = Lr[r];
+        if (MODE == SIGMOID && active && a.d.head_bias) hbx[x] = a.d.head_bias[hx[x]];
     }
     const int cw = active ? (hbeg + rb / QT) / rep - gc0 : 0;   // the warp's key/value group among the CTA's
     float mrun[2] = {-INFINITY, -INFINITY}, lrun[2] = {0.f, 0.f};
@@ -244,6 +248,10 @@ __global__ void __launch_bounds__(NT) mix_tc_kernel(MixArgs a) {
                     const bool ok = okx[x] && col < nk && j <= posx[x] && j >= lox[x];
                     float v = s[n][e] * a.d.scale;
                     if (a.dist_bias && ok) v += a.dist_bias[(long long)min(posx[x] - j, a.far) * H + hx[x]];
+                    if (MODE == SIGMOID) {
+                        s[n][e] = ok ? __fdividef(1.f, 1.f + __expf(-(v + hbx[x]))) : 0.f;
+                        continue;
+                    }
                     v = ok ? v : -INFINITY;
                     if (!APPLY || ONE) {
                         s[n][e] = v;
@@ -409,31 +417,32 @@ __global__ void __launch_bounds__(NT) mix_tc_kernel(MixArgs a) {
     }
 }
 
-template <int KT, int NDV, bool APPLY, bool TALK, bool ONE>
+template <int KT, int NDV, bool APPLY, bool TALK, int MODE>
 int launch_tc(const MixArgs& a, dim3 grid, size_t smem, cudaStream_t stream) {
     static PerDeviceOnce once;
     if (once.need())
-        ASD_CUDA(cudaFuncSetAttribute(mix_tc_kernel<KT, NDV, APPLY, TALK, ONE>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+        ASD_CUDA(cudaFuncSetAttribute(mix_tc_kernel<KT, NDV, APPLY, TALK, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                       220 * 1024));
-    mix_tc_kernel<KT, NDV, APPLY, TALK, ONE><<<grid, NT, smem, stream>>>(a);
+    mix_tc_kernel<KT, NDV, APPLY, TALK, MODE><<<grid, NT, smem, stream>>>(a);
     count_launch(1);
     ASD_CUDA(cudaGetLastError());
     return 0;
 }
 
 template <int KT, int NDV>
-int launch_apply(const MixArgs& a, bool one, dim3 grid, size_t smem, cudaStream_t stream) {
-    if (a.talk) return launch_tc<KT, NDV, true, true, false>(a, grid, smem, stream);
-    return one ? launch_tc<KT, NDV, true, false, true>(a, grid, smem, stream)
-               : launch_tc<KT, NDV, true, false, false>(a, grid, smem, stream);
+int launch_apply(const MixArgs& a, int mode, dim3 grid, size_t smem, cudaStream_t stream) {
+    if (a.talk) return launch_tc<KT, NDV, true, true, TWO_PASS>(a, grid, smem, stream);
+    if (mode == SIGMOID) return launch_tc<KT, NDV, true, false, SIGMOID>(a, grid, smem, stream);
+    return mode == ONLINE ? launch_tc<KT, NDV, true, false, ONLINE>(a, grid, smem, stream)
+                          : launch_tc<KT, NDV, true, false, TWO_PASS>(a, grid, smem, stream);
 }
 
 template <int KT>
-int launch_passes(const MixArgs& a, bool one, int ndv, dim3 grid, size_t smem_stats, size_t smem_apply, cudaStream_t stream) {
-    if (!one && launch_tc<KT, 4, false, false, false>(a, grid, smem_stats, stream)) return -1;
-    return ndv == 4 ? launch_apply<KT, 4>(a, one, grid, smem_apply, stream)
-                    : (ndv == 8 ? launch_apply<KT, 8>(a, one, grid, smem_apply, stream)
-                                : launch_apply<KT, 16>(a, one, grid, smem_apply, stream));
+int launch_passes(const MixArgs& a, int mode, int ndv, dim3 grid, size_t smem_stats, size_t smem_apply, cudaStream_t stream) {
+    if (mode == TWO_PASS && launch_tc<KT, 4, false, false, TWO_PASS>(a, grid, smem_stats, stream)) return -1;
+    return ndv == 4 ? launch_apply<KT, 4>(a, mode, grid, smem_apply, stream)
+                    : (ndv == 8 ? launch_apply<KT, 8>(a, mode, grid, smem_apply, stream)
+                                : launch_apply<KT, 16>(a, mode, grid, smem_apply, stream));
 }
 
 }  // namespace
@@ -476,16 +485,17 @@ int launch_mix_attention_tc(MixArgs a, int nseq, int max_qlen, int max_kv_len, c
         shares = (int)std::min<long long>((296 + base - 1) / base, (long long)std::max(1, key_tiles / 2));
         shares = std::min(shares, 32);
         while (shares > 1 && ((long long)shares * a.ix.M * H * dv > ws.part_elems ||
-                              (long long)2 * shares * a.ix.M * H > ws.stats_elems))
+                              (!a.d.sigmoid && (long long)2 * shares * a.ix.M * H > ws.stats_elems)))
             --shares;
     }
-    if (!ws.stats || (long long)2 * shares * a.ix.M * H > ws.stats_elems) return 1;
+    if (!a.d.sigmoid && (!ws.stats || (long long)2 * shares * a.ix.M * H > ws.stats_elems)) return 1;
     a.shares = shares;
     const size_t smem_stats = (size_t)tc_layout(gp * rep * QT, DS, VS, gp, KT, H, false, false, pipe ? 2 : 1).total;
     const dim3 grid(tiles, nseq, shares * ngroups);
-    const bool one = !talk && shares == 1;      // no mix across heads and one share: one pass with a running maximum
-    const int rc = KT == 64 ? launch_passes<64>(a, one, ndv, grid, smem_stats, smem_apply, stream)
-                            : launch_passes<32>(a, one, ndv, grid, smem_stats, smem_apply, stream);
+    // no mix across heads and one share: one pass with a running maximum
+    const int mode = a.d.sigmoid ? SIGMOID : (!talk && shares == 1 ? ONLINE : TWO_PASS);
+    const int rc = KT == 64 ? launch_passes<64>(a, mode, ndv, grid, smem_stats, smem_apply, stream)
+                            : launch_passes<32>(a, mode, ndv, grid, smem_stats, smem_apply, stream);
     if (rc) return -1;
     if (shares > 1 && launch_mix_merge(a, stream)) return -1;
     return 0;

@@ -1,5 +1,6 @@
 // Mixture-of-experts routing: fp32 softmax over all experts, the `top` largest probabilities kept as gates (as they
-// are, or divided by their sum, which is the softmax over the chosen logits alone), then the (token, choice) pairs grouped by expert so that each expert's rows are contiguous
+// are, or divided by their sum, which is the softmax over the chosen logits alone), or sigmoid scores chosen with a
+// correction among the best groups of experts; then the (token, choice) pairs grouped by expert so that each expert's rows are contiguous
 // for the grouped linear layers.  Which slot inside an expert's group a pair gets does not matter for the result: every
 // slot is computed on its own and a token's choices are summed in choice order by the layer close.
 #include <cuda_runtime.h>
@@ -13,13 +14,105 @@ namespace asd {
 
 namespace {
 
+struct RouteChoice {
+    int top, renorm, sigmoid, groups, keep;
+    const float* correction;
+    float scale;
+};
+
+// One warp chooses a token's experts from its logits z[E] and writes their indices and gates; counts take one each.
+// pr: E floats of scratch; gr: c.groups floats of scratch (used with groups > 1 only).
+__device__ void choose_experts(const float* z, int E, const RouteChoice& c, float* pr, float* gr, int* expert_of, float* gate,
+                               int* counts, int lane) {
+    const float TAKEN = -INFINITY;
+    float inv = 1.f;
+    if (c.sigmoid) {
+        for (int e = lane; e < E; e += 32) pr[e] = 1.f / (1.f + expf(-z[e])) + (c.correction ? c.correction[e] : 0.f);
+        __syncwarp();
+        if (c.groups > 1) {
+            const int n = E / c.groups;
+            for (int g = lane; g < c.groups; g += 32) {
+                float a = -INFINITY, b = -INFINITY;      // the two largest choice scores of the group
+                for (int e = g * n; e < (g + 1) * n; ++e) {
+                    const float v = pr[e];
+                    if (v > a) {
+                        b = a;
+                        a = v;
+                    } else if (v > b) {
+                        b = v;
+                    }
+                }
+                gr[g] = n > 1 ? a + b : a;
+            }
+            __syncwarp();
+            // a group stays if fewer than `keep` groups stand before it (larger score, or equal and lower index)
+            for (int g = lane; g < c.groups; g += 32) {
+                int before = 0;
+                for (int o = 0; o < c.groups; ++o) before += gr[o] > gr[g] || (gr[o] == gr[g] && o < g);
+                if (before >= c.keep)
+                    for (int e = g * n; e < (g + 1) * n; ++e) pr[e] = TAKEN;
+            }
+        }
+    } else {
+        float mx = -INFINITY;
+        for (int e = lane; e < E; e += 32) mx = fmaxf(mx, z[e]);
+        mx = warp_max(mx);
+        float s = 0.f;
+        for (int e = lane; e < E; e += 32) {
+            const float v = expf(z[e] - mx);
+            pr[e] = v;
+            s += v;
+        }
+        inv = 1.f / warp_sum(s);
+    }
+    float chosen = 0.f;
+    __syncwarp();
+    for (int k = 0; k < c.top; ++k) {
+        float best = TAKEN;
+        int bi = 0x7fffffff;
+        for (int e = lane; e < E; e += 32) {
+            const float v = pr[e];
+            if (v > best) {        // increasing e per lane: the first maximum wins
+                best = v;
+                bi = e;
+            }
+        }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+            const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+            if (ob > best || (ob == best && oi < bi)) {
+                best = ob;
+                bi = oi;
+            }
+        }
+        if (bi >= E) bi = k;       // no comparable score is left (NaN logits): any expert, its gate is NaN as well
+        if (lane == 0) {
+            const float s = c.sigmoid ? 1.f / (1.f + expf(-z[bi])) : pr[bi];
+            expert_of[k] = bi;
+            gate[k] = s * inv;
+            chosen += s;
+            atomicAdd(&counts[bi], 1);
+            pr[bi] = TAKEN;
+        }
+        __syncwarp();
+    }
+    if (lane == 0 && c.sigmoid) {
+        const float r = c.scale / (chosen + 1e-20f);
+        for (int k = 0; k < c.top; ++k) gate[k] *= r;
+    } else if (lane == 0 && c.renorm) {   // gates over the chosen alone: e^(z - max) / sum of the chosen e^(z - max)
+        const float r = 1.f / (chosen * inv);
+        for (int k = 0; k < c.top; ++k) gate[k] *= r;
+    }
+}
+
 // one warp per token; probs of the token live in shared memory (E floats per warp).  With x != nullptr the warp first
 // computes the token's router logits itself, z[e] = sum_d x[m][d] * wr[e][d] in fp32 (lane-strided partial sums in
 // increasing d, then the fixed warp tree: the same for a token whatever else is in the batch), eight experts per pass
 // over the row.
 __global__ void moe_route_kernel(const float* logits, const void* x, int xf32, const void* wr, int wf32, int D, float* z_out,
-                                 int M, int E, int top, int* expert_of, float* gate, int* counts, const float* bias,
-                                 int renorm) {
+                                 int M, int E, int zld, RouteChoice c, int* expert_of, float* gate, int* counts,
+                                 const float* bias) {
     extern __shared__ float sm[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int m = blockIdx.x * (blockDim.x >> 5) + warp;
@@ -49,113 +142,27 @@ __global__ void moe_route_kernel(const float* logits, const void* x, int xf32, c
         }
         __syncwarp();
     }
-    const float* z = x ? zs : logits + (long long)m * E;
-    float mx = -INFINITY;
-    for (int e = lane; e < E; e += 32) mx = fmaxf(mx, z[e]);
-    mx = warp_max(mx);
-    float s = 0.f;
-    for (int e = lane; e < E; e += 32) {
-        const float v = expf(z[e] - mx);
-        pr[e] = v;
-        s += v;
-    }
-    s = warp_sum(s);
-    const float inv = 1.f / s;
-    float chosen = 0.f;
-    __syncwarp();
-    for (int k = 0; k < top; ++k) {
-        float best = -1.f;
-        int bi = 0x7fffffff;
-        for (int e = lane; e < E; e += 32) {
-            const float v = pr[e];
-            if (v > best) {        // increasing e per lane: the first maximum wins
-                best = v;
-                bi = e;
-            }
-        }
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) {
-            const float ob = __shfl_xor_sync(0xffffffffu, best, o);
-            const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
-            if (ob > best || (ob == best && oi < bi)) {
-                best = ob;
-                bi = oi;
-            }
-        }
-        if (lane == 0) {
-            expert_of[(long long)m * top + k] = bi;
-            gate[(long long)m * top + k] = best * inv;
-            chosen += best;
-            atomicAdd(&counts[bi], 1);
-            pr[bi] = -2.f;         // taken
-        }
-        __syncwarp();
-    }
-    if (renorm && lane == 0) {   // gates over the chosen alone: e^(z - max) / sum of the chosen e^(z - max)
-        const float r = 1.f / (chosen * inv);
-        for (int k = 0; k < top; ++k) gate[(long long)m * top + k] *= r;
-    }
+    const float* z = x ? zs : logits + (long long)m * zld;
+    choose_experts(z, E, c, pr, zs, expert_of + (long long)m * c.top, gate + (long long)m * c.top, counts, lane);
 }
 
 // Few tokens (M * top <= 4096): choice, group sizes, offsets and scatter in ONE CTA with shared-memory counters, so that a
 // decode step spends two launches on routing (logits, then this) instead of five.
-__global__ void __launch_bounds__(256) moe_route_small_kernel(const float* logits, int M, int E, int top, int* expert_of,
-                                                              float* gate, int* group_off, int* sorted_tok, int* slot_of,
-                                                              int renorm) {
+__global__ void __launch_bounds__(256) moe_route_small_kernel(const float* logits, int M, int E, int zld, RouteChoice c,
+                                                              int* expert_of, float* gate, int* group_off, int* sorted_tok,
+                                                              int* slot_of) {
     extern __shared__ float sm[];
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
-    int* cnt = reinterpret_cast<int*>(sm + (size_t)nw * E);     // [E] group sizes, then fill counters
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5, top = c.top;
+    const int per = E + (c.groups > 1 ? c.groups : 0);
+    int* cnt = reinterpret_cast<int*>(sm + (size_t)nw * per);   // [E] group sizes, then fill counters
     int* off = cnt + E;                                          // [E + 1]
     for (int e = threadIdx.x; e < E; e += blockDim.x) cnt[e] = 0;
     __syncthreads();
-    float* pr = sm + (size_t)warp * E;
+    float* pr = sm + (size_t)warp * per;
     for (int m = warp; m < M; m += nw) {
-        const float* z = logits + (long long)m * E;
-        float mx = -INFINITY;
-        for (int e = lane; e < E; e += 32) mx = fmaxf(mx, z[e]);
-        mx = warp_max(mx);
-        float s = 0.f;
-        for (int e = lane; e < E; e += 32) {
-            const float v = expf(z[e] - mx);
-            pr[e] = v;
-            s += v;
-        }
-        s = warp_sum(s);
-        const float inv = 1.f / s;
-        float chosen = 0.f;
+        choose_experts(logits + (long long)m * zld, E, c, pr, pr + E, expert_of + (long long)m * top,
+                       gate + (long long)m * top, cnt, lane);
         __syncwarp();
-        for (int k = 0; k < top; ++k) {
-            float best = -1.f;
-            int bi = 0x7fffffff;
-            for (int e = lane; e < E; e += 32) {
-                const float v = pr[e];
-                if (v > best) {
-                    best = v;
-                    bi = e;
-                }
-            }
-#pragma unroll
-            for (int o = 16; o > 0; o >>= 1) {
-                const float ob = __shfl_xor_sync(0xffffffffu, best, o);
-                const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
-                if (ob > best || (ob == best && oi < bi)) {
-                    best = ob;
-                    bi = oi;
-                }
-            }
-            if (lane == 0) {
-                expert_of[(long long)m * top + k] = bi;
-                gate[(long long)m * top + k] = best * inv;
-                chosen += best;
-                atomicAdd(&cnt[bi], 1);
-                pr[bi] = -2.f;
-            }
-            __syncwarp();
-        }
-        if (renorm && lane == 0) {
-            const float r = 1.f / (chosen * inv);
-            for (int k = 0; k < top; ++k) gate[(long long)m * top + k] *= r;
-        }
     }
     __syncthreads();
     if (threadIdx.x == 0) {
@@ -180,11 +187,12 @@ __global__ void __launch_bounds__(256) moe_route_small_kernel(const float* logit
 
 // router logits, one CTA per token: z[m][e] = sum_d x[m][d] * wr[e][d] in fp32.  Thread t sums d = t, t + 128, ... in
 // increasing order, then the fixed warp tree and the warps in index order: a token's logits do not depend on the batch.
+// rows >= E: rows beyond the experts' are computed alike (no bias); z_out rows are `rows` floats.
 __global__ void __launch_bounds__(128) moe_logits_kernel(const void* x, int xf32, const void* wr, int wf32, int D, int E,
-                                                         float* z_out, const float* bias) {
+                                                         int rows, float* z_out, const float* bias) {
     __shared__ float red[4][8];
     const int m = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    for (int e0 = 0; e0 < E; e0 += 8) {
+    for (int e0 = 0; e0 < rows; e0 += 8) {
         float acc[8];
 #pragma unroll
         for (int j = 0; j < 8; ++j) acc[j] = 0.f;
@@ -193,7 +201,7 @@ __global__ void __launch_bounds__(128) moe_logits_kernel(const void* x, int xf32
             const float xv = ldx(x, (long long)m * D + d, xf32);
 #pragma unroll
             for (int j = 0; j < 8; ++j)
-                if (e0 + j < E) acc[j] = fmaf(xv, ldx(wr, (long long)(e0 + j) * D + d, wf32), acc[j]);
+                if (e0 + j < rows) acc[j] = fmaf(xv, ldx(wr, (long long)(e0 + j) * D + d, wf32), acc[j]);
         }
         __syncthreads();
 #pragma unroll
@@ -202,10 +210,10 @@ __global__ void __launch_bounds__(128) moe_logits_kernel(const void* x, int xf32
             if (lane == 0) red[warp][j] = v;
         }
         __syncthreads();
-        if (threadIdx.x < 8 && e0 + threadIdx.x < E)
-            z_out[(long long)m * E + e0 + threadIdx.x] =
+        if (threadIdx.x < 8 && e0 + threadIdx.x < rows)
+            z_out[(long long)m * rows + e0 + threadIdx.x] =
                 (((red[0][threadIdx.x] + red[1][threadIdx.x]) + red[2][threadIdx.x]) + red[3][threadIdx.x]) +
-                (bias ? bias[e0 + threadIdx.x] : 0.f);
+                (bias && e0 + threadIdx.x < E ? bias[e0 + threadIdx.x] : 0.f);
     }
 }
 
@@ -239,25 +247,33 @@ int launch_moe_route(const float* logits, const MoeRouterInput* in, int M, int E
     if (E <= 0 || top <= 0 || top > E) return set_error("moe: need 0 < top <= experts (top %d, experts %d)", top, E);
     if ((size_t)E * 8 * sizeof(float) > 48 * 1024) return set_error("moe: more than 1536 experts");
     if (!logits && !in) return set_error("moe: neither logits nor router inputs");
-    const int renorm = in ? in->renorm : 0;
-    if (in && in->logits_out && (long long)M * top <= 4096 && (size_t)(8 * E + 2 * E + 1) * 4 <= 48 * 1024) {
-        moe_logits_kernel<<<M, 128, 0, stream>>>(in->x, in->x_f32, in->w, in->w_f32, in->D, E, in->logits_out, in->bias);
-        moe_route_small_kernel<<<1, 256, (size_t)(8 * E + 2 * E + 1) * sizeof(float), stream>>>(
-            in->logits_out, M, E, top, expert_of, gate, group_off, sorted_tok, slot_of, in->renorm);
+    RouteChoice c{top, 0, 0, 1, 1, nullptr, 1.f};
+    if (in) c = RouteChoice{top, in->renorm, in->sigmoid, in->groups, in->keep, in->correction, in->scale};
+    if (c.sigmoid) {
+        if (!in->logits_out) return set_error("moe: sigmoid scores need logits_out");
+        if (c.groups < 1 || E % c.groups || c.keep < 1 || c.keep > c.groups || top > c.keep * (E / c.groups))
+            return set_error("moe: %d experts in %d groups, %d kept, %d chosen", E, c.groups, c.keep, top);
+    }
+    const int zld = E + (in ? in->extra : 0);
+    const size_t small_smem = (size_t)(8 * (E + (c.groups > 1 ? c.groups : 0)) + 2 * E + 1) * sizeof(float);
+    if (in && in->logits_out && (long long)M * top <= 4096 && small_smem <= 48 * 1024) {
+        moe_logits_kernel<<<M, 128, 0, stream>>>(in->x, in->x_f32, in->w, in->w_f32, in->D, E, zld, in->logits_out, in->bias);
+        moe_route_small_kernel<<<1, 256, small_smem, stream>>>(in->logits_out, M, E, zld, c, expert_of, gate, group_off,
+                                                               sorted_tok, slot_of);
         count_launch(2);
         ASD_CUDA(cudaGetLastError());
         return 0;
     }
     ASD_CUDA(cudaMemsetAsync(counters, 0, sizeof(int) * E, stream));
     if (in && in->logits_out) {          // a CTA per token for the logits: few tokens still spread over the GPU
-        moe_logits_kernel<<<M, 128, 0, stream>>>(in->x, in->x_f32, in->w, in->w_f32, in->D, E, in->logits_out, in->bias);
+        moe_logits_kernel<<<M, 128, 0, stream>>>(in->x, in->x_f32, in->w, in->w_f32, in->D, E, zld, in->logits_out, in->bias);
         count_launch(1);
         logits = in->logits_out;
         in = nullptr;
     }
     moe_route_kernel<<<(M + 3) / 4, 128, (size_t)E * 8 * sizeof(float), stream>>>(
         logits, in ? in->x : nullptr, in ? in->x_f32 : 0, in ? in->w : nullptr, in ? in->w_f32 : 0, in ? in->D : 0,
-        nullptr, M, E, top, expert_of, gate, counters, in ? in->bias : nullptr, renorm);
+        nullptr, M, E, zld, c, expert_of, gate, counters, in ? in->bias : nullptr);
     moe_offsets_kernel<<<1, 32, 0, stream>>>(counters, group_off, E);
     const int n = M * top;
     moe_scatter_kernel<<<(n + 255) / 256, 256, 0, stream>>>(expert_of, n, top, E, group_off, counters, sorted_tok, slot_of);

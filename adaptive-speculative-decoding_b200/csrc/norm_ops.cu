@@ -26,6 +26,23 @@ __global__ void embed_scaled_kernel(SeqIndex ix, const void* embed, int wf32, fl
     }
 }
 
+// x[m] = embed[token] * scale + (sin at even, cos at odd coordinates of position * freq[coordinate / 2]).  The angle is
+// brought into one turn in fp64, so that a far position's angle is as exact as a near one's.
+__global__ void embed_sinusoid_kernel(SeqIndex ix, const void* embed, int wf32, float scale, const double* freq, float* x,
+                                      int D) {
+    const int m = blockIdx.x;
+    const long long src = (long long)ix.tokens[m] * D, dst = (long long)m * D;
+    const double pos = (double)ix.positions[m];
+    constexpr double TURN = 6.283185307179586476925;
+    for (int i = threadIdx.x; 2 * i < D; i += blockDim.x) {
+        const double a = pos * freq[i];
+        float sn, cs;
+        sincosf((float)(a - TURN * rint(a / TURN)), &sn, &cs);
+        x[dst + 2 * i] = fmaf(ldx(embed, src + 2 * i, wf32), scale, sn);
+        if (2 * i + 1 < D) x[dst + 2 * i + 1] = fmaf(ldx(embed, src + 2 * i + 1, wf32), scale, cs);
+    }
+}
+
 constexpr int MAX_NORM_GROUPS = 64;   // parts a grouped norm may split a row into
 
 // dynamic shared memory: D floats (the row being built) + 33 for the block sums + MAX_NORM_GROUPS group factors
@@ -38,36 +55,53 @@ __global__ void row_close_kernel(RowClose c) {
     const long long base = (long long)m * D;
     const long long in_base = c.rows ? (long long)c.rows[m] * D : base;
     const float off = c.plain_w ? 0.f : 1.f;
-    float post = 1.f;
-    if (c.y && c.post_w) {
+    auto inv_rms = [&](const float* src) {
         float ss = 0.f;
         for (int d = threadIdx.x; d < D; d += blockDim.x) {
-            const float v = c.y[base + d];
+            const float v = src[base + d];
             ss += v * v;
         }
-        post = 1.f / sqrtf(block_sum(ss, red) / (float)D + c.eps);
-    }
+        return 1.f / sqrtf(block_sum(ss, red) / (float)D + c.eps);
+    };
+    const float post = c.y && c.post_w ? inv_rms(c.y) * c.y_scale : 1.f;
+    const float post2 = c.y2 ? inv_rms(c.y2) * c.y_scale : 1.f;
+    const float ff_gate = c.ff_gate ? 1.f / (1.f + expf(-c.ff_gate[(long long)m * c.ff_gate_ld])) : 1.f;
 #pragma unroll 4
     for (int d = threadIdx.x; d < D; d += blockDim.x) {
-        float v = c.x_in ? c.x_in[in_base + d] : 0.f;
+        float v = 0.f;
+        const float xv = c.x_in ? c.x_in[in_base + d] : 0.f;
+        if (c.mult == 1.f) v = xv;
         if (c.y) v += c.post_w ? c.y[base + d] * post * (off + c.post_w[d]) : c.y[base + d];
+        if (c.y2) v += c.y2[base + d] * post2 * (off + c.post_w2[d]);
+        if (c.ff) v = fmaf(ff_gate, c.ff[base + d], v);
         for (int k = 0; k < c.top; ++k)     // routed experts' results in choice order
             v = fmaf(c.gate[(long long)m * c.top + k], c.expert_out[(long long)c.slot_of[(long long)m * c.top + k] * D + d], v);
         if (c.bias) v += c.bias[d];
+        if (c.mult != 1.f) v = fmaf(c.mult, v, xv);
         row[d] = v;
         if (c.x_out) c.x_out[base + d] = v;
     }
     if (c.next_w) {
         __syncthreads();
+        float mean = 0.f;
+        if (c.next_b) {
+            float t = 0.f;
+            for (int d = threadIdx.x; d < D; d += blockDim.x) t += row[d];
+            mean = block_sum(t, red) / (float)D;
+        }
         for (int g = 0; g < G; ++g) {
             float ss = 0.f;
-            for (int d = g * Dg + threadIdx.x; d < (g + 1) * Dg; d += blockDim.x) ss += row[d] * row[d];
+            for (int d = g * Dg + threadIdx.x; d < (g + 1) * Dg; d += blockDim.x) ss += (row[d] - mean) * (row[d] - mean);
             const float t = block_sum(ss, red);
             if (threadIdx.x == 0) gs[g] = 1.f / sqrtf(t / (float)Dg + c.eps);
         }
         __syncthreads();
-        for (int d = threadIdx.x; d < D; d += blockDim.x)
-            stx(c.hn, base + d, c.hn_f32, row[d] * gs[d / Dg] * (off + c.next_w[d]));
+        for (int d = threadIdx.x; d < D; d += blockDim.x) {
+            float v = (row[d] - mean) * gs[d / Dg] * (off + c.next_w[d]);
+            if (c.next_b) v += c.next_b[d];
+            stx(c.hn, base + d, c.hn_f32, v);
+            if (c.hn_copy) c.hn_copy[base + d] = v;
+        }
     } else if (c.cat) {
         for (int d = threadIdx.x; d < D; d += blockDim.x) {
             stx(c.hn, 2 * base + d, c.hn_f32, row[d]);
@@ -178,11 +212,22 @@ int launch_embed_scaled(const SeqIndex& ix, const void* embed, int wf32, float s
     return 0;
 }
 
+int launch_embed_sinusoid(const SeqIndex& ix, const void* embed, int wf32, float scale, const double* freq, float* x, int D,
+                          cudaStream_t stream) {
+    if (ix.M <= 0) return 0;
+    embed_sinusoid_kernel<<<ix.M, row_threads(D), 0, stream>>>(ix, embed, wf32, scale, freq, x, D);
+    count_launch(1);
+    ASD_CUDA(cudaGetLastError());
+    return 0;
+}
+
 int launch_row_close(const RowClose& c, cudaStream_t stream) {
     if (c.M <= 0) return 0;
     if (c.D <= 0 || ((c.next_w || c.cat) && !c.hn)) return set_error("row_close: bad arguments");
     if (c.groups <= 0 || c.groups > MAX_NORM_GROUPS || c.D % c.groups)
         return set_error("row_close: %d norm groups do not divide width %d (at most %d)", c.groups, c.D, MAX_NORM_GROUPS);
+    if (c.next_b && c.groups != 1) return set_error("row_close: a layer norm has no groups");
+    if (c.y2 && !c.post_w2) return set_error("row_close: the second branch has no norm weight");
     if (c.top > 0 && (!c.expert_out || !c.slot_of || !c.gate)) return set_error("row_close: expert results missing");
     const size_t smem = (size_t)(c.D + 33 + MAX_NORM_GROUPS) * sizeof(float);
     if (smem > 200 * 1024) return set_error("row_close: width %d does not fit shared memory", c.D);

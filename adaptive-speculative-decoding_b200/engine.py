@@ -10,7 +10,7 @@ from typing import Dict, Optional
 
 import torch
 
-from ._lib import (AsdError, LukopelConfigC, LukopelLayerC, MavipelConfigC, MavipelLayerC, MezilixConfigC, MezilixLayerC, ModelConfigC, RivetarConfigC,
+from ._lib import (AsdError, DikopelConfigC, DikopelLayerC, LukopelConfigC, LukopelLayerC, MavipelConfigC, MavipelLayerC, MezilixConfigC, MezilixLayerC, ModelConfigC, RivetarConfigC,
                    RivetarLayerC, check, lib)
 from .models.qwen2 import Qwen2Config, pack_layer, random_packed_layer
 from .ops import NUM_FEATURES
@@ -791,6 +791,36 @@ class LukopelEngine(RivetarEngine):
             arr[i] = LukopelLayerC(l.heads, l.kv_heads, l.dim, l.vdim, 0 if full else 1, 1 if full else 0,
                                    1 if full else 0, l.chunk, l.far if full else 0, l.temp_every if full else 0,
                                    1 if l.ff_kind else 0, l.ff, l.scale, l.temp_coef if full else 0.0)
+        return c, arr
+
+
+class DikopelEngine(RivetarEngine):
+    """One Dikopel-family model on one GPU: wraps an ``asd_dikopel_engine_t`` handle.  Same ownership as
+    ``RivetarEngine``: per layer (also one that uses another layer's weights) the paged key/value cache of a parallel
+    layer's attention (``PageTable``) and, in one fp32 buffer, the carried inputs of the convolutions and the recurrent
+    states, one entry per ring position; entry position % ring is the state after that position, and a forward that
+    starts a slot at position 0 starts from zero, so reused slots carry nothing over.  Same ``forward`` interface as
+    ``QwenEngine``, so ``SpecDecoder``, ``Stage`` and the trace runner drive it unchanged."""
+
+    TYPE_CODE = {"mlstm": 0, "parallel": 1}
+    FF_CODE = {None: 0, "dense": 1, "moe": 2}
+    PREFIX = "dikopel"
+    PROFILE_CLASSES = ("dense", "attention", "recurrence", "experts", "router", "activation", "glue", "lm_head")
+
+    @staticmethod
+    def _family():
+        from .models import dikopel
+        return dikopel
+
+    def _c_config(self, cfg, max_tokens: int, page_size: int, dtype):
+        c = DikopelConfigC(cfg.width, cfg.vocab_size, cfg.num_hidden_layers, cfg.eps, cfg.embed_scale, cfg.residual_mult,
+                           cfg.input_taps, max_tokens, page_size, self.ring, 1 if dtype == torch.float32 else 0)
+        arr = (DikopelLayerC * max(1, cfg.num_hidden_layers))()
+        for i, l in enumerate(cfg.layers):
+            arr[i] = DikopelLayerC(self.TYPE_CODE[l.type], l.weights_of, l.heads, l.dim, l.vdim, l.a_heads, l.a_kv_heads,
+                                   l.a_dim, l.a_vdim, l.r_heads, l.r_kv_heads, l.r_dim, l.r_vdim, l.conv,
+                                   self.FF_CODE[l.ff_kind], l.ff, l.experts, l.top, l.expert_ff, l.shared_ff, l.groups,
+                                   l.keep, l.gate_cap, l.scale, l.router_scale)
         return c, arr
 
 

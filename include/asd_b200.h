@@ -540,6 +540,86 @@ ASD_API int asd_lukopel_forward(asd_lukopel_engine_t* e, const int32_t* tokens, 
 ASD_API int asd_lukopel_profile_read(asd_lukopel_engine_t* e, float* ms_by_class, int* launches_by_class, int nclass);
 ASD_API int asd_lukopel_device_error(asd_lukopel_engine_t* e);
 
+/* ------------------------------------------------------------------------------------------------------------------
+ * Dikopel family engine (dikopel_engine.cu).  x = embed[token] * embed_scale + sinusoids of the position (sin(p *
+ * 10000^(-2i/width)) at 2i, cos of the same at 2i + 1).  Every layer has ONE norm whose result both sublayers read:
+ * h = norm1(x); x <- x + residual_mult * (mixer(h + conv(h)) + ff(h)), where conv is a causal convolution over time per
+ * channel with input_taps taps.  logits = head . final_norm(x).  Norms are layer norms with weight and bias (eps inside the
+ * root).  A layer's mixer is
+ *   type 0  matrix memory with exponential gates: q (times dim^(-1/2)), k (heads x dim), v (heads x vdim), logarithmic gates
+ *           i = gate_cap tanh(. / gate_cap), f = log_sigmoid(gate_cap tanh(. / gate_cap)) per head with biases; running
+ *           maximum M (starts at 0), M' = max(f + M, i), S <- exp(f + M - M') S + exp(i - M') k v^T, n likewise with k alone,
+ *           o = S^T q / (max(|n . q|, exp(-M')) + 1e-6); o / rms(o) per head * out_norm[heads * vdim] * sigmoid(gate), then
+ *           the output projection;
+ *   type 1  two mixers on the same input; their results are RMS-normed over the width (weights out_left, out_right) and
+ *           averaged.  Left: grouped-query causal attention (a_heads, a_kv_heads, a_dim, a_vdim) whose weights are
+ *           sigmoid(scale * q . k + head_bias[head]), not normalised over the keys.  Right: gated delta rule: q, k
+ *           (r_kv_heads x r_dim) and v (r_heads x r_vdim) pass a causal convolution over time (conv taps per channel) and
+ *           silu, q and k become unit vectors, q times r_dim^(-1/2); beta = sigmoid per head; one decay per head and
+ *           position g = exp(-exp(a_log) softplus(. + dt_bias)); S <- g S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q;
+ *           o / rms(o) * out_norm[r_vdim] * silu(gate), then the output projection.
+ * ff_kind 0: none; 1: W_down (silu(W_gate h) * W_up h); 2: `experts` such layers of size expert_ff of which every token
+ * takes `top`: scores s = sigmoid(router logits, fp32), choice by s + correction among the experts of the `keep` best of
+ * `groups` groups of neighbours (a group's score: the sum of its two largest choice scores), weights s / (sum of the chosen
+ * s + 1e-20) * router_scale; plus a shared expert of size shared_ff times sigmoid(its gate row . h) (0: none).
+ * weights_of >= 0: the layer uses that layer's tensors (all its other fields equal that layer's) with a cache and state of
+ * its own; -1: tensors of its own.
+ *
+ * dtype as for the Rivetar engine.  Paged pool: per layer of type 1 [num_pages][page_size][a_kv_heads * (a_dim + a_vdim)],
+ * keys then values, layers back to back.  State (caller allocated, fp32), per layer: carried rows of the input convolution
+ * [max_seqs][input_taps - 1 + ring - 1][width], carried inputs of the mixer's convolution [max_seqs][conv - 1 + ring - 1]
+ * [channels] (type 1), then the recurrent state [max_seqs][ring] x (type 0: S [heads][dim][vdim], then for every head and
+ * block of 32 value columns n [dim] and M; type 1: [r_heads][r_dim][r_vdim]); entry position % ring holds the state AFTER
+ * that position, so a caller may re-feed any of the last `ring` positions; a run that starts at position 0 starts from zero.
+ */
+typedef struct asd_dikopel_layer_config {
+    int type;                                                 /* 0 matrix memory, 1 sigmoid attention + gated delta rule */
+    int weights_of;
+    int heads, dim, vdim;                                                    /* type 0 */
+    int a_heads, a_kv_heads, a_dim, a_vdim;                                  /* type 1, left */
+    int r_heads, r_kv_heads, r_dim, r_vdim, conv;                            /* type 1, right */
+    int ff_kind, ff, experts, top, expert_ff, shared_ff, groups, keep;
+    float gate_cap, scale, router_scale;
+} asd_dikopel_layer_config;
+typedef struct asd_dikopel_config {
+    int width, vocab, n_layers;
+    float eps, embed_scale, residual_mult;
+    int input_taps;
+    int max_tokens, page_size, ring, dtype;
+} asd_dikopel_config;
+typedef struct asd_dikopel_engine asd_dikopel_engine_t;
+
+ASD_API asd_dikopel_engine_t* asd_dikopel_create(const asd_dikopel_config* cfg, const asd_dikopel_layer_config* layers);
+ASD_API void asd_dikopel_destroy(asd_dikopel_engine_t* e);
+/* Weights by name; matrices row-major [out, in] in the engine's dtype, vectors and everything marked fp32 always fp32.
+ * layer -1: "embed" [vocab, width], "final_norm", "final_norm_b" [width], "head" [vocab, width].  Every layer with tensors of
+ * its own: "norm1", "norm1_b" [width], "input_conv" fp32 [width][input_taps], "w_in" = the matrices that read the mixer
+ * input stacked by rows, "w_o" = the output projection:
+ *   type 0: w_in [q | k | v | gate | input gate | forget gate]; also "i_bias", "f_bias" [heads], "out_norm" [heads * vdim];
+ *   type 1: w_in [left q | k | v | right q | k | v | gate | beta | decay], w_o the left and "w_o2" the right output
+ *           projection; also "head_bias" [a_heads], "conv_w" fp32 [right q, k, v channels][conv], "a_log", "dt_bias"
+ *           [r_heads], "out_norm" [r_vdim], "out_left", "out_right" [width].
+ * ff_kind 1: "w_gu" [2 ff, width] (gate rows, then up rows), "w_down" [width, ff].  ff_kind 2: "router" fp32 [experts (+ 1:
+ * the shared expert's gate row), width], "correction" [experts], "w_egu" [experts][2 expert_ff, width], "w_edown"
+ * [experts][width, expert_ff], and with a shared expert "w_sgu" [2 shared_ff, width], "w_sdown" [width, shared_ff]. */
+ASD_API int asd_dikopel_set_tensor(asd_dikopel_engine_t* e, int layer, const char* name, const void* data);
+ASD_API size_t asd_dikopel_cache_bytes(const asd_dikopel_engine_t* e, int num_pages);
+ASD_API size_t asd_dikopel_state_bytes(const asd_dikopel_engine_t* e, int max_seqs);
+ASD_API int asd_dikopel_set_cache(asd_dikopel_engine_t* e, void* pool, int num_pages, const int32_t* page_table,
+                                  int max_seqs, int max_pages_per_seq, float* state);
+/* options: "tc_linear", "tc_min_rows" as for the Mezilix engine; "attn_general" as for the Lukopel engine; "profile" */
+ASD_API int asd_dikopel_set_option(asd_dikopel_engine_t* e, const char* name, int value);
+/* Same arguments as asd_engine_forward (M <= max_tokens).  layer_out (optional, fp32 [n_layers][M][width]) receives the
+ * stream that leaves every layer. */
+ASD_API int asd_dikopel_forward(asd_dikopel_engine_t* e, const int32_t* tokens, const int32_t* positions,
+                                const int32_t* token_slot, int M, const int32_t* cu_q, const int32_t* seq_slot, int nseq,
+                                int max_qlen, int max_kv_len, const int32_t* logit_rows, int n_logit_rows,
+                                float* logits_out, long long logits_ld, float* layer_out, void* stream);
+/* ms and launches by kernel class since the last read (nclass >= 8): 0 dense projections, 1 attention, 2 recurrences,
+ * 3 expert layers, 4 router, 5 feed-forward activations, 6 embedding / norms / convolutions / cache append, 7 output head */
+ASD_API int asd_dikopel_profile_read(asd_dikopel_engine_t* e, float* ms_by_class, int* launches_by_class, int nclass);
+ASD_API int asd_dikopel_device_error(asd_dikopel_engine_t* e);
+
 #ifdef __cplusplus
 }
 #endif
