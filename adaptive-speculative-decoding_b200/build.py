@@ -29,7 +29,8 @@ COMPONENTS = {
     "mezilix": ["mezilix_engine.cu", "stream_ops.cu"],
     "rivetar": ["rivetar_engine.cu", "gla.cu", "window_attention.cu"],
     "delta": ["delta_rule.cu"],                 # delta rules and short convolutions
-    "mixattn": ["mixed_attention.cu", "mixed_attention_tc.cu", "sigmoid_attention.cu"],
+    "mixattn": ["mixed_attention.cu", "mixed_attention_tc.cu", "sigmoid_attention.cu",
+                "sigmoid_attention_tc.cu"],
     "mavipel": ["mavipel_engine.cu", "talking_attention.cu"],
     "lukopel": ["lukopel_engine.cu", "residual_streams.cu"],
     "dikopel": ["dikopel_engine.cu", "mlstm.cu"],

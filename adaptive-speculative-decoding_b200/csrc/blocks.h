@@ -431,7 +431,8 @@ int launch_mix_post(const SeqIndex& ix, float* qkv, long long ld, const MixDims&
 int mix_attention_check(const MixDims& d, int talk);
 // Workspace: stats fp32 [2][shares][M][heads] (maximum and sum of every key share), part fp32 [shares][M][heads * dv].
 // scores fp32 [M][heads][keys] of steps of few tokens (optional).  mode 0: steps of few tokens and, in a bf16 engine,
-// prompts on the tensor cores take kernels of their own; 1: everything runs the general CUDA-core kernels.
+// prompts on the tensor cores take kernels of their own; 1: everything runs the general CUDA-core kernels; 2: steps of few
+// tokens stay on the CUDA cores.
 struct MixWork {
     float* stats = nullptr;
     float* part = nullptr;
@@ -470,13 +471,13 @@ struct MlstmInput {
     const float* bias_i = nullptr;   // [heads]
     const float* bias_f = nullptr;
 };
-// floats of state per sequence and ring entry: heads * (dk * dv + ceil(dv / 32) * (dk + 1))
+// floats of state per sequence and ring entry: heads * (dk * dv + ceil(dv / 32) * (dk + 1)), rounded up to a multiple of 4
 size_t mlstm_state_elems(const MlstmDims& d);
 // state fp32 [slots][ring][ S [heads][dk][dv] | [heads][ceil(dv / 32)] x (n [dk], M) ]; entry position % ring holds the state after that
 // position.  A sequence whose first new position is 0 starts from zero, any other from entry (position - 1) % ring; the
 // last `ring` new positions of a sequence store theirs.  out fp32 [M][heads * dv].
-int launch_mlstm_recurrence(const SeqIndex& ix, const int* cu_q, const int* seq_slot, int nseq, const MlstmInput& in,
-                            const MlstmDims& d, float* state, int ring, float* out, cudaStream_t stream);
+int launch_mlstm_recurrence(const SeqIndex& ix, const int* cu_q, const int* seq_slot, int nseq, int max_qlen,
+                            const MlstmInput& in, const MlstmDims& d, float* state, int ring, float* out, cudaStream_t stream);
 
 int preload_blocks();
 

@@ -127,8 +127,8 @@ static int mix_mlstm(DkEngine* e, const DkLayer& ly, const DkRun& run, int li, c
         MlstmInput in;
         in.q = e->proj, in.k = e->proj + nk, in.v = e->proj + 2 * nk, in.zi = e->proj + 2 * (nk + nv), in.zf = in.zi + c.heads;
         in.ld = ly.ld_in, in.bias_i = ly.f("i_bias"), in.bias_f = ly.f("f_bias");
-        if (launch_mlstm_recurrence(b.ix, b.cu_q, b.seq_slot, b.nseq, in, mlstm_dims(c), e->state + run.state_off, e->c.ring,
-                                    e->orec, s))
+        if (launch_mlstm_recurrence(b.ix, b.cu_q, b.seq_slot, b.nseq, b.max_qlen, in, mlstm_dims(c),
+                                    e->state + run.state_off, e->c.ring, e->orec, s))
             return -1;
     }
     {
@@ -333,6 +333,14 @@ static size_t pool_elems(const DkEngine* e, const DkRun& r, int num_pages) {
     return (n + 7) & ~(size_t)7;
 }
 
+// the parts of one layer's carried state, floats per sequence slot count; every part starts on a 16-byte boundary
+static size_t up4(size_t n) { return (n + 3) & ~(size_t)3; }
+static size_t input_floats(const DkEngine* e, int max_seqs) { return up4((size_t)max_seqs * e->input_ring * e->c.width); }
+static size_t conv_floats(const DkLayer& ly, int max_seqs) { return up4((size_t)max_seqs * ly.conv_elems); }
+static size_t state_floats(const DkEngine* e, const DkLayer& ly, int max_seqs) {
+    return up4((size_t)max_seqs * e->c.ring * ly.state_elems);
+}
+
 static const char* const kLayerNames[] = {"norm1", "norm1_b", "input_conv", "w_in", "w_o", "w_o2", "i_bias", "f_bias",
                                           "out_norm", "head_bias", "conv_w", "a_log", "dt_bias", "out_left", "out_right",
                                           "w_gu", "w_down", "router", "correction", "w_egu", "w_edown", "w_sgu", "w_sdown"};
@@ -532,7 +540,7 @@ size_t asd_dikopel_state_bytes(const asd_dikopel_engine_t* h, int max_seqs) {
     size_t n = 0;
     for (const DkRun& r : e->runs) {
         const DkLayer& ly = e->layers[r.layer];
-        n += (size_t)max_seqs * ((size_t)e->input_ring * e->c.width + ly.conv_elems + (size_t)e->c.ring * ly.state_elems);
+        n += input_floats(e, max_seqs) + conv_floats(ly, max_seqs) + state_floats(e, ly, max_seqs);
     }
     return n * sizeof(float);
 }
@@ -551,11 +559,11 @@ int asd_dikopel_set_cache(asd_dikopel_engine_t* h, void* pool, int num_pages, co
         r.cache_off = off;
         off += pool_elems(e, r, num_pages);
         r.input_off = soff;
-        soff += (size_t)max_seqs * e->input_ring * e->c.width;
+        soff += input_floats(e, max_seqs);
         r.conv_off = soff;
-        soff += (size_t)max_seqs * ly.conv_elems;
+        soff += conv_floats(ly, max_seqs);
         r.state_off = soff;
-        soff += (size_t)max_seqs * e->c.ring * ly.state_elems;
+        soff += state_floats(e, ly, max_seqs);
     }
     return 0;
 }
@@ -573,7 +581,7 @@ int asd_dikopel_set_option(asd_dikopel_engine_t* h, const char* name, int value)
         return 0;
     }
     if (!strcmp(name, "attn_general")) {
-        e->attn_ws.mode = value ? 1 : 0;
+        e->attn_ws.mode = value;
         return 0;
     }
     if (!strcmp(name, "profile")) {

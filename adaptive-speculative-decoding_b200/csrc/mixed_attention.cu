@@ -836,6 +836,10 @@ int launch_mix_attention(const SeqIndex& ix, const int* cu_q, const int* seq_slo
     a.QT = 1, a.shares = 1, a.gp = 1, a.rag = 1;
     a.vec = (d.dk % 4 == 0 && d.dv % 4 == 0) ? 1 : 0;
     // steps of few tokens; prompts of a bf16 engine on the tensor cores; else (and for sizes those refuse) the CUDA cores
+    if (d.sigmoid && max_qlen < 8 && ws.mode == 0) {
+        const int rc = launch_sigmoid_attention_decode_tc(a, nseq, max_qlen, max_kv_len, ws, stream);
+        if (rc <= 0) return rc;
+    }
     if (max_qlen <= 4 && ws.mode != 1) {
         const int rc = d.sigmoid ? launch_sigmoid_attention_decode(a, max_kv_len, ws, stream)
                                  : launch_mix_attention_decode(a, nseq, max_kv_len, ws, stream);

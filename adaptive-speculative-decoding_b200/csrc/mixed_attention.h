@@ -37,6 +37,9 @@ int launch_mix_attention_tc(MixArgs a, int nseq, int max_qlen, int max_kv_len, c
 int launch_mix_attention_decode(MixArgs a, int nseq, int max_kv_len, const MixWork& ws, cudaStream_t stream);
 // The same with sigmoid weights (sigmoid_attention.cu): one pass.  Same returns.
 int launch_sigmoid_attention_decode(MixArgs a, int max_kv_len, const MixWork& ws, cudaStream_t stream);
+// And on the tensor cores for bf16 cache rows (sigmoid_attention_tc.cu).  Same returns.
+int launch_sigmoid_attention_decode_tc(MixArgs a, int nseq, int max_qlen, int max_kv_len, const MixWork& ws,
+                                       cudaStream_t stream);
 // sums the key shares' partial results in index order, applies the gates, writes the engine's element type
 int launch_mix_merge(const MixArgs& a, cudaStream_t stream);
 

@@ -44,7 +44,7 @@ struct MlstmArgs {
 
 // every block of 32 value columns keeps its own copy of n and M, so that CTAs share no state
 __host__ __device__ inline size_t entry_elems(const MlstmDims& d) {
-    return (size_t)d.heads * ((size_t)d.dk * d.dv + (size_t)((d.dv + 31) / 32) * (d.dk + 1));
+    return ((size_t)d.heads * ((size_t)d.dk * d.dv + (size_t)((d.dv + 31) / 32) * (d.dk + 1)) + 3) & ~(size_t)3;
 }
 
 // shared memory in floats: two buffers of { q [CH][dkp], k [CH][dkp], v [CH][32], zi [CH], zf [CH] }; then per chunk
@@ -219,17 +219,112 @@ __global__ void __launch_bounds__(MAXT, 1) mlstm_recurrence_kernel(MlstmArgs a) 
     }
 }
 
+// Steps of one token per sequence: the state is read and written once, so a CTA streams a (sequence, head)'s rows, four
+// columns a thread and eight rows in flight, up to 128 columns wide.
+constexpr int ST = 256, SCOLS = 128, SU = 8;
+__global__ void __launch_bounds__(ST) mlstm_step_kernel(MlstmArgs a) {
+    extern __shared__ __align__(16) float sm[];
+    const int seq = blockIdx.x, head = blockIdx.y, col0 = blockIdx.z * SCOLS, tid = threadIdx.x;
+    const int m = a.cu_q[seq];
+    if (m >= a.cu_q[seq + 1]) return;
+    const int dk = a.d.dk, dv = a.d.dv, H = a.d.heads, ring = a.ring;
+    const int L = (min(SCOLS, dv - col0)) >> 2, R = ST / L;      // threads per row, rows per pass
+    const int rg = tid / L, c4 = (tid - rg * L) * 4;
+    const int pos = a.ix.positions[m];
+    const size_t entry = entry_elems(a.d);
+    float* slot = a.state + (size_t)a.seq_slot[seq] * ring * entry;
+    const float* src = slot + (size_t)((pos + ring - 1) % ring) * entry;      // pos - 1, not read at position 0
+    float* dst = slot + (size_t)(pos % ring) * entry;
+    const size_t st_S = (size_t)head * dk * dv + col0 + c4;
+    const bool old = pos > 0, live = rg < R;
+    float* qs = sm;
+    float* ks = qs + dk;
+    float* red = ks + dk;             // [R][4 L] partial results, then 33 for a block sum
+    float4 S[SU];
+    auto load = [&](int r0) {
+#pragma unroll
+        for (int u = 0; u < SU; ++u) {
+            const int r = r0 + u * R;
+            S[u] = (live && old && r < dk) ? *reinterpret_cast<const float4*>(src + st_S + (size_t)r * dv)
+                                           : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+    };
+    load(rg);
+    const long long row = (long long)m * a.in.ld;
+    for (int i = tid; i < dk; i += ST) {
+        qs[i] = a.in.q[row + (long long)head * dk + i];
+        ks[i] = a.in.k[row + (long long)head * dk + i];
+    }
+    const int nb = (dv + 31) / 32, b0 = col0 / 32, b1 = min(nb, b0 + SCOLS / 32);
+    const size_t st_n = (size_t)H * dk * dv + ((size_t)head * nb) * (dk + 1);
+    const float mold = old ? src[st_n + (size_t)b0 * (dk + 1) + dk] : 0.f;
+    const float cap = a.d.cap;
+    const float li = cap * tanhf((a.in.zi[row + head] + (a.in.bias_i ? a.in.bias_i[head] : 0.f)) / cap);
+    const float lf = log_sigmoid(cap * tanhf((a.in.zf[row + head] + (a.in.bias_f ? a.in.bias_f[head] : 0.f)) / cap));
+    const float mnew = fmaxf(lf + mold, li);
+    const float keep = expf(lf + mold - mnew), put = expf(li - mnew), flr = expf(-mnew);
+    float pv[4] = {0.f, 0.f, 0.f, 0.f}, o[4] = {0.f, 0.f, 0.f, 0.f};
+    if (live)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) pv[e] = put * a.in.v[row + (long long)head * dv + col0 + c4 + e];
+    __syncthreads();
+    for (int r0 = rg; r0 < dk && live; r0 += SU * R) {
+        if (r0 != rg) load(r0);
+#pragma unroll
+        for (int u = 0; u < SU; ++u) {
+            const int r = r0 + u * R;
+            if (r >= dk) break;
+            const float kk = ks[r], qq = qs[r];
+            float4 s = S[u];
+            s.x = fmaf(kk, pv[0], keep * s.x), s.y = fmaf(kk, pv[1], keep * s.y);
+            s.z = fmaf(kk, pv[2], keep * s.z), s.w = fmaf(kk, pv[3], keep * s.w);
+            *reinterpret_cast<float4*>(dst + st_S + (size_t)r * dv) = s;
+            o[0] = fmaf(s.x, qq, o[0]), o[1] = fmaf(s.y, qq, o[1]);
+            o[2] = fmaf(s.z, qq, o[2]), o[3] = fmaf(s.w, qq, o[3]);
+        }
+    }
+    float nq = 0.f;
+    for (int i = tid; i < (b1 - b0) * dk; i += ST) {      // the copies of n that belong to these columns
+        const int j = i / dk, r = i - j * dk;
+        const size_t at = st_n + (size_t)(b0 + j) * (dk + 1) + r;
+        const float n = fmaf(ks[r], put, old ? keep * src[at] : 0.f);
+        dst[at] = n;
+        if (j == 0) nq = fmaf(n, qs[r], nq);
+    }
+    if (live)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) red[rg * 4 * L + c4 + e] = o[e];
+    nq = block_sum(nq, red + R * 4 * L) * a.d.q_scale;     // its barriers also complete red, and every read of M
+    if (tid < b1 - b0) dst[st_n + (size_t)(b0 + tid) * (dk + 1) + dk] = mnew;
+    const float inv = a.d.q_scale / (fmaxf(fabsf(nq), flr) + 1e-6f);
+    for (int c = tid; c < 4 * L; c += ST) {
+        float t = 0.f;
+        for (int r = 0; r < R; ++r) t += red[r * 4 * L + c];
+        a.out[(long long)m * H * dv + (long long)head * dv + col0 + c] = t * inv;
+    }
+}
+
 }  // namespace
 
 size_t mlstm_state_elems(const MlstmDims& d) { return entry_elems(d); }
 
-int launch_mlstm_recurrence(const SeqIndex& ix, const int* cu_q, const int* seq_slot, int nseq, const MlstmInput& in,
-                            const MlstmDims& d, float* state, int ring, float* out, cudaStream_t stream) {
+int launch_mlstm_recurrence(const SeqIndex& ix, const int* cu_q, const int* seq_slot, int nseq, int max_qlen,
+                            const MlstmInput& in, const MlstmDims& d, float* state, int ring, float* out, cudaStream_t stream) {
     if (ix.M <= 0 || nseq <= 0) return 0;
     if (d.heads <= 0 || d.dv <= 0 || d.dk <= 0 || d.dk > 1024) return set_error("mlstm: key size %d outside 1..1024", d.dk);
     if (!(d.cap > 0.f)) return set_error("mlstm: the gate cap must be positive");
     if (ring <= 0 || !state) return set_error("mlstm: no state");
     if (!in.q || !in.k || !in.v || !in.zi || !in.zf) return set_error("mlstm: missing inputs");
+    if (max_qlen == 1 && d.dv % 4 == 0 && (reinterpret_cast<uintptr_t>(state) & 15) == 0 && d.heads <= 65535) {
+        MlstmArgs a;
+        a.ix = ix, a.cu_q = cu_q, a.seq_slot = seq_slot, a.in = in, a.d = d, a.state = state, a.ring = ring, a.CH = 1;
+        a.v16 = 0, a.out = out;
+        const size_t smem = (size_t)(2 * d.dk + 4 * ST + 33) * sizeof(float);
+        mlstm_step_kernel<<<dim3(nseq, d.heads, (d.dv + SCOLS - 1) / SCOLS), ST, smem, stream>>>(a);
+        count_launch(1);
+        ASD_CUDA(cudaGetLastError());
+        return 0;
+    }
     int rows = 4;
     while (rows < 32 && rows * 4 < d.dk) rows *= 2;     // four warps up to key size 128, then more
     const int RS = (d.dk + rows - 1) / rows, dkp = RS * rows;

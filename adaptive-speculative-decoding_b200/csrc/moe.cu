@@ -185,35 +185,47 @@ __global__ void __launch_bounds__(256) moe_route_small_kernel(const float* logit
     }
 }
 
-// router logits, one CTA per token: z[m][e] = sum_d x[m][d] * wr[e][d] in fp32.  Thread t sums d = t, t + 128, ... in
+// router logits, one CTA per token (or four): z[m][e] = sum_d x[m][d] * wr[e][d] in fp32.  Thread t sums d = t, t + 128, ... in
 // increasing order, then the fixed warp tree and the warps in index order: a token's logits do not depend on the batch.
 // rows >= E: rows beyond the experts' are computed alike (no bias); z_out rows are `rows` floats.
-__global__ void __launch_bounds__(128) moe_logits_kernel(const void* x, int xf32, const void* wr, int wf32, int D, int E,
+// NJ rows of w and NTOK tokens share a pass (the sums and their order do not depend on either).
+template <int NJ, int NTOK>
+__global__ void __launch_bounds__(128) moe_logits_kernel(const void* x, int xf32, const void* wr, int wf32, int D, int M, int E,
                                                          int rows, float* z_out, const float* bias) {
-    __shared__ float red[4][8];
-    const int m = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    for (int e0 = 0; e0 < rows; e0 += 8) {
-        float acc[8];
+    __shared__ float red[4][NTOK][NJ];
+    const int m0 = blockIdx.x * NTOK, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    for (int e0 = 0; e0 < rows; e0 += NJ) {
+        float acc[NTOK][NJ];
 #pragma unroll
-        for (int j = 0; j < 8; ++j) acc[j] = 0.f;
-#pragma unroll 4
+        for (int t = 0; t < NTOK; ++t)
+#pragma unroll
+            for (int j = 0; j < NJ; ++j) acc[t][j] = 0.f;
+#pragma unroll(NTOK > 1 ? 2 : 4)
         for (int d = threadIdx.x; d < D; d += 128) {
-            const float xv = ldx(x, (long long)m * D + d, xf32);
+            float xv[NTOK];
 #pragma unroll
-            for (int j = 0; j < 8; ++j)
-                if (e0 + j < rows) acc[j] = fmaf(xv, ldx(wr, (long long)(e0 + j) * D + d, wf32), acc[j]);
+            for (int t = 0; t < NTOK; ++t) xv[t] = m0 + t < M ? ldx(x, (long long)(m0 + t) * D + d, xf32) : 0.f;
+#pragma unroll
+            for (int j = 0; j < NJ; ++j)
+                if (e0 + j < rows) {
+                    const float w = ldx(wr, (long long)(e0 + j) * D + d, wf32);
+#pragma unroll
+                    for (int t = 0; t < NTOK; ++t) acc[t][j] = fmaf(xv[t], w, acc[t][j]);
+                }
         }
         __syncthreads();
 #pragma unroll
-        for (int j = 0; j < 8; ++j) {
-            const float v = warp_sum(acc[j]);
-            if (lane == 0) red[warp][j] = v;
-        }
+        for (int t = 0; t < NTOK; ++t)
+#pragma unroll
+            for (int j = 0; j < NJ; ++j) {
+                const float v = warp_sum(acc[t][j]);
+                if (lane == 0) red[warp][t][j] = v;
+            }
         __syncthreads();
-        if (threadIdx.x < 8 && e0 + threadIdx.x < rows)
-            z_out[(long long)m * rows + e0 + threadIdx.x] =
-                (((red[0][threadIdx.x] + red[1][threadIdx.x]) + red[2][threadIdx.x]) + red[3][threadIdx.x]) +
-                (bias && e0 + threadIdx.x < E ? bias[e0 + threadIdx.x] : 0.f);
+        const int t = threadIdx.x / NJ, j = threadIdx.x % NJ;
+        if (t < NTOK && m0 + t < M && e0 + j < rows)
+            z_out[(long long)(m0 + t) * rows + e0 + j] =
+                (((red[0][t][j] + red[1][t][j]) + red[2][t][j]) + red[3][t][j]) + (bias && e0 + j < E ? bias[e0 + j] : 0.f);
     }
 }
 
@@ -239,6 +251,20 @@ __global__ void moe_scatter_kernel(const int* expert_of, int n, int top, int E, 
     slot_of[i] = slot;
 }
 
+template <int NJ, int NTOK>
+void launch_logits_as(const MoeRouterInput& in, int M, int E, int rows, cudaStream_t stream) {
+    moe_logits_kernel<NJ, NTOK><<<(M + NTOK - 1) / NTOK, 128, 0, stream>>>(in.x, in.x_f32, in.w, in.w_f32, in.D, M, E, rows,
+                                                                         in.logits_out, in.bias);
+}
+void launch_logits(const MoeRouterInput& in, int M, int E, int rows, cudaStream_t stream) {
+    if (M >= 1024)        // enough CTAs without one per token: each row of w is read for four tokens
+        launch_logits_as<8, 4>(in, M, E, rows, stream);
+    else if (rows <= 8)
+        launch_logits_as<8, 1>(in, M, E, rows, stream);
+    else
+        launch_logits_as<16, 1>(in, M, E, rows, stream);
+}
+
 }  // namespace
 
 int launch_moe_route(const float* logits, const MoeRouterInput* in, int M, int E, int top, int* expert_of, float* gate,
@@ -257,7 +283,7 @@ int launch_moe_route(const float* logits, const MoeRouterInput* in, int M, int E
     const int zld = E + (in ? in->extra : 0);
     const size_t small_smem = (size_t)(8 * (E + (c.groups > 1 ? c.groups : 0)) + 2 * E + 1) * sizeof(float);
     if (in && in->logits_out && (long long)M * top <= 4096 && small_smem <= 48 * 1024) {
-        moe_logits_kernel<<<M, 128, 0, stream>>>(in->x, in->x_f32, in->w, in->w_f32, in->D, E, zld, in->logits_out, in->bias);
+        launch_logits(*in, M, E, zld, stream);
         moe_route_small_kernel<<<1, 256, small_smem, stream>>>(in->logits_out, M, E, zld, c, expert_of, gate, group_off,
                                                                sorted_tok, slot_of);
         count_launch(2);
@@ -266,7 +292,7 @@ int launch_moe_route(const float* logits, const MoeRouterInput* in, int M, int E
     }
     ASD_CUDA(cudaMemsetAsync(counters, 0, sizeof(int) * E, stream));
     if (in && in->logits_out) {          // a CTA per token for the logits: few tokens still spread over the GPU
-        moe_logits_kernel<<<M, 128, 0, stream>>>(in->x, in->x_f32, in->w, in->w_f32, in->D, E, zld, in->logits_out, in->bias);
+        launch_logits(*in, M, E, zld, stream);
         count_launch(1);
         logits = in->logits_out;
         in = nullptr;

@@ -68,7 +68,7 @@ class DikopelLayer:
     def state_elems(self) -> int:
         """floats of recurrent state per sequence (and ring entry)"""
         if self.type == "mlstm":
-            return self.heads * (self.dim * self.vdim + (self.vdim + 31) // 32 * (self.dim + 1))
+            return (self.heads * (self.dim * self.vdim + (self.vdim + 31) // 32 * (self.dim + 1)) + 3) // 4 * 4
         return self.r_heads * self.r_dim * self.r_vdim
 
     @property

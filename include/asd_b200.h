@@ -569,7 +569,8 @@ ASD_API int asd_lukopel_device_error(asd_lukopel_engine_t* e);
  * keys then values, layers back to back.  State (caller allocated, fp32), per layer: carried rows of the input convolution
  * [max_seqs][input_taps - 1 + ring - 1][width], carried inputs of the mixer's convolution [max_seqs][conv - 1 + ring - 1]
  * [channels] (type 1), then the recurrent state [max_seqs][ring] x (type 0: S [heads][dim][vdim], then for every head and
- * block of 32 value columns n [dim] and M; type 1: [r_heads][r_dim][r_vdim]); entry position % ring holds the state AFTER
+ * block of 32 value columns n [dim] and M, rounded up to a multiple of 4; type 1: [r_heads][r_dim][r_vdim]), every one of
+ * these parts starting on a 16-byte boundary; entry position % ring holds the state AFTER
  * that position, so a caller may re-feed any of the last `ring` positions; a run that starts at position 0 starts from zero.
  */
 typedef struct asd_dikopel_layer_config {
