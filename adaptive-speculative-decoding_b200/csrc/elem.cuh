@@ -24,6 +24,17 @@ __device__ __forceinline__ void stf<__nv_bfloat16>(__nv_bfloat16* p, float v) {
 __device__ __forceinline__ float ldx(const void* p, long long i, int f32) {
     return f32 ? ((const float*)p)[i] : __bfloat162float(((const __nv_bfloat16*)p)[i]);
 }
+// four consecutive elements from a place that is a multiple of four in a 16-byte aligned buffer
+__device__ __forceinline__ void ldx4(const void* p, long long i, int f32, float (&v)[4]) {
+    if (f32) {
+        const float4 f = *reinterpret_cast<const float4*>((const float*)p + i);
+        v[0] = f.x, v[1] = f.y, v[2] = f.z, v[3] = f.w;
+    } else {
+        const uint2 r = *reinterpret_cast<const uint2*>((const __nv_bfloat16*)p + i);
+        v[0] = __uint_as_float(r.x << 16), v[1] = __uint_as_float(r.x & 0xffff0000u);
+        v[2] = __uint_as_float(r.y << 16), v[3] = __uint_as_float(r.y & 0xffff0000u);
+    }
+}
 __device__ __forceinline__ void stx(void* p, long long i, int f32, float v) {
     if (f32)
         ((float*)p)[i] = v;

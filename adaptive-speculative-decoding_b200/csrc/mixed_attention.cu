@@ -721,11 +721,32 @@ __global__ void mix_post_kernel(SeqIndex ix, float* qkv, long long ld, MixDims d
     }
 }
 
+// nothing to do but the append: the queries stay as they are
+template <typename T>
+__global__ void mix_append_kernel(SeqIndex ix, const float* qkv, long long ld, int nq, int n, PagedRows cache) {
+    const int m = blockIdx.x, pos = ix.positions[m], slot = ix.token_slot[m];
+    const int page = cache.page_table[(long long)slot * cache.max_pages + pos / cache.page_size];
+    T* dst = static_cast<T*>(cache.pool) + ((long long)page * cache.page_size + pos % cache.page_size) * n;
+    const float* src = qkv + (long long)m * ld + nq;
+#pragma unroll 4
+    for (int i = threadIdx.x; i < n; i += blockDim.x) stf(dst + i, src[i]);
+}
+
 }  // namespace
 
 int launch_mix_post(const SeqIndex& ix, float* qkv, long long ld, const MixDims& d, const MixPost& p,
                     const PagedRows& cache, cudaStream_t stream) {
     if (ix.M <= 0) return 0;
+    if (!p.bias && !p.q_norm && !p.k_norm && !p.temp_every && !p.head_factor && !p.v_unit) {
+        const int nq = d.heads * d.dk, nkv = d.kv_heads * (d.dk + d.dv), threads = nkv >= 1024 ? 256 : 128;
+        if (cache.f32)
+            mix_append_kernel<float><<<ix.M, threads, 0, stream>>>(ix, qkv, ld, nq, nkv, cache);
+        else
+            mix_append_kernel<__nv_bfloat16><<<ix.M, threads, 0, stream>>>(ix, qkv, ld, nq, nkv, cache);
+        count_launch(1);
+        ASD_CUDA(cudaGetLastError());
+        return 0;
+    }
     const int n = d.heads * d.dk + d.kv_heads * (d.dk + d.dv), units = d.heads + 2 * d.kv_heads;
     const size_t smem = (size_t)(n + units) * sizeof(float);
     if (smem > 200 * 1024) return set_error("mix_post: a row of %d values does not fit shared memory", n);

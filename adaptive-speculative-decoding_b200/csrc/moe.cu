@@ -185,13 +185,13 @@ __global__ void __launch_bounds__(256) moe_route_small_kernel(const float* logit
     }
 }
 
-// router logits, one CTA per token (or four): z[m][e] = sum_d x[m][d] * wr[e][d] in fp32.  Thread t sums d = t, t + 128, ... in
+// router logits, one CTA per token (or four): z[m][e] = sum_d x[m][d] * wr[e][d] in fp32.  Thread t sums blocks of four elements t, t + 128, ... in
 // increasing order, then the fixed warp tree and the warps in index order: a token's logits do not depend on the batch.
 // rows >= E: rows beyond the experts' are computed alike (no bias); z_out rows are `rows` floats.
 // NJ rows of w and NTOK tokens share a pass (the sums and their order do not depend on either).
 template <int NJ, int NTOK>
 __global__ void __launch_bounds__(128) moe_logits_kernel(const void* x, int xf32, const void* wr, int wf32, int D, int M, int E,
-                                                         int rows, float* z_out, const float* bias) {
+                                                         int rows, float* z_out, const float* bias, int vec) {
     __shared__ float red[4][NTOK][NJ];
     const int m0 = blockIdx.x * NTOK, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     for (int e0 = 0; e0 < rows; e0 += NJ) {
@@ -200,18 +200,31 @@ __global__ void __launch_bounds__(128) moe_logits_kernel(const void* x, int xf32
         for (int t = 0; t < NTOK; ++t)
 #pragma unroll
             for (int j = 0; j < NJ; ++j) acc[t][j] = 0.f;
-#pragma unroll(NTOK > 1 ? 2 : 4)
-        for (int d = threadIdx.x; d < D; d += 128) {
-            float xv[NTOK];
+        // four consecutive elements per load; a row that is no multiple of four ends element by element
+        const int D4 = vec ? D >> 2 : 0;
+#pragma unroll 2
+        for (int i = threadIdx.x; i < D4; i += 128) {
+            float xv[NTOK][4];
 #pragma unroll
-            for (int t = 0; t < NTOK; ++t) xv[t] = m0 + t < M ? ldx(x, (long long)(m0 + t) * D + d, xf32) : 0.f;
+            for (int t = 0; t < NTOK; ++t) ldx4(x, (long long)(m0 + t < M ? m0 + t : m0) * D + 4 * i, xf32, xv[t]);
 #pragma unroll
-            for (int j = 0; j < NJ; ++j)
-                if (e0 + j < rows) {
-                    const float w = ldx(wr, (long long)(e0 + j) * D + d, wf32);
+            for (int j = 0; j < NJ; ++j) {      // beyond the last row: its product again, not stored (no branch between loads)
+                float w[4];
+                ldx4(wr, (long long)min(e0 + j, rows - 1) * D + 4 * i, wf32, w);
 #pragma unroll
-                    for (int t = 0; t < NTOK; ++t) acc[t][j] = fmaf(xv[t], w, acc[t][j]);
-                }
+                for (int t = 0; t < NTOK; ++t)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) acc[t][j] = fmaf(xv[t][e], w[e], acc[t][j]);
+            }
+        }
+        for (int d = 4 * D4 + threadIdx.x; d < D; d += 128) {
+#pragma unroll
+            for (int t = 0; t < NTOK; ++t) {
+                const float xv = ldx(x, (long long)(m0 + t < M ? m0 + t : m0) * D + d, xf32);
+#pragma unroll
+                for (int j = 0; j < NJ; ++j)
+                    if (e0 + j < rows) acc[t][j] = fmaf(xv, ldx(wr, (long long)(e0 + j) * D + d, wf32), acc[t][j]);
+            }
         }
         __syncthreads();
 #pragma unroll
@@ -253,16 +266,24 @@ __global__ void moe_scatter_kernel(const int* expert_of, int n, int top, int E, 
 
 template <int NJ, int NTOK>
 void launch_logits_as(const MoeRouterInput& in, int M, int E, int rows, cudaStream_t stream) {
+    const uintptr_t at = reinterpret_cast<uintptr_t>(in.x) | reinterpret_cast<uintptr_t>(in.w);
+    const int vec = in.D % 4 == 0 && (at & 15) == 0;
     moe_logits_kernel<NJ, NTOK><<<(M + NTOK - 1) / NTOK, 128, 0, stream>>>(in.x, in.x_f32, in.w, in.w_f32, in.D, M, E, rows,
-                                                                         in.logits_out, in.bias);
+                                                                         in.logits_out, in.bias, vec);
 }
+// the passes over a token's row are few and even
 void launch_logits(const MoeRouterInput& in, int M, int E, int rows, cudaStream_t stream) {
-    if (M >= 1024)        // enough CTAs without one per token: each row of w is read for four tokens
-        launch_logits_as<8, 4>(in, M, E, rows, stream);
-    else if (rows <= 8)
-        launch_logits_as<8, 1>(in, M, E, rows, stream);
-    else
-        launch_logits_as<16, 1>(in, M, E, rows, stream);
+    if (M >= 1024) {      // enough CTAs without one per token: each row of w is read for four tokens
+        const int per = (rows + (rows + 11) / 12 - 1) / ((rows + 11) / 12);
+        if (per <= 8) return launch_logits_as<8, 4>(in, M, E, rows, stream);
+        if (per <= 10) return launch_logits_as<10, 4>(in, M, E, rows, stream);
+        return launch_logits_as<12, 4>(in, M, E, rows, stream);
+    }
+    const int per = (rows + (rows + 15) / 16 - 1) / ((rows + 15) / 16);
+    if (per <= 8) return launch_logits_as<8, 1>(in, M, E, rows, stream);
+    if (per <= 10) return launch_logits_as<10, 1>(in, M, E, rows, stream);
+    if (per <= 12) return launch_logits_as<12, 1>(in, M, E, rows, stream);
+    return launch_logits_as<16, 1>(in, M, E, rows, stream);
 }
 
 }  // namespace

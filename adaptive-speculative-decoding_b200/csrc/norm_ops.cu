@@ -45,41 +45,105 @@ __global__ void embed_sinusoid_kernel(SeqIndex ix, const void* embed, int wf32, 
 
 constexpr int MAX_NORM_GROUPS = 64;   // parts a grouped norm may split a row into
 
-// dynamic shared memory: D floats (the row being built) + 33 for the block sums + MAX_NORM_GROUPS group factors
+template <int V>
+__device__ __forceinline__ void loadv(const float* p, float (&v)[V]) {
+    if constexpr (V == 4) {
+        const float4 f = *reinterpret_cast<const float4*>(p);
+        v[0] = f.x, v[1] = f.y, v[2] = f.z, v[3] = f.w;
+    } else {
+        v[0] = *p;
+    }
+}
+template <int V>
+__device__ __forceinline__ void storev(float* p, const float (&v)[V]) {
+    if constexpr (V == 4)
+        *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+    else
+        *p = v[0];
+}
+template <int V>
+__device__ __forceinline__ void storevx(void* p, long long i, int f32, const float (&v)[V]) {
+    if (V == 4 && !f32) {
+        __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[V > 1 ? 1 : 0]), hi = __floats2bfloat162_rn(v[V > 2 ? 2 : 0], v[V - 1]);
+        *reinterpret_cast<uint2*>((__nv_bfloat16*)p + i) =
+            make_uint2(*reinterpret_cast<uint32_t*>(&lo), *reinterpret_cast<uint32_t*>(&hi));
+    } else if (f32) {
+        storev<V>((float*)p + i, v);
+    } else {
+        stx(p, i, 0, v[0]);
+    }
+}
+
+// dynamic shared memory: D floats (the row being built) + 33 for the block sums + MAX_NORM_GROUPS group factors.  V
+// consecutive elements per thread and step: 4 where width, norm groups and addresses allow, else 1.
+template <int V>
 __global__ void row_close_kernel(RowClose c) {
-    extern __shared__ float sm[];
+    extern __shared__ __align__(16) float sm[];
     float* row = sm;
     float* red = sm + c.D;
     float* gs = red + 33;
-    const int m = blockIdx.x, D = c.D, G = c.groups, Dg = D / G;
+    const int m = blockIdx.x, D = c.D, G = c.groups, Dg = D / G, step = blockDim.x * V, first = threadIdx.x * V;
     const long long base = (long long)m * D;
     const long long in_base = c.rows ? (long long)c.rows[m] * D : base;
     const float off = c.plain_w ? 0.f : 1.f;
     auto inv_rms = [&](const float* src) {
         float ss = 0.f;
-        for (int d = threadIdx.x; d < D; d += blockDim.x) {
-            const float v = src[base + d];
-            ss += v * v;
+        for (int d = first; d < D; d += step) {
+            float v[V];
+            loadv<V>(src + base + d, v);
+#pragma unroll
+            for (int e = 0; e < V; ++e) ss += v[e] * v[e];
         }
         return 1.f / sqrtf(block_sum(ss, red) / (float)D + c.eps);
     };
     const float post = c.y && c.post_w ? inv_rms(c.y) * c.y_scale : 1.f;
     const float post2 = c.y2 ? inv_rms(c.y2) * c.y_scale : 1.f;
     const float ff_gate = c.ff_gate ? 1.f / (1.f + expf(-c.ff_gate[(long long)m * c.ff_gate_ld])) : 1.f;
-#pragma unroll 4
-    for (int d = threadIdx.x; d < D; d += blockDim.x) {
-        float v = 0.f;
-        const float xv = c.x_in ? c.x_in[in_base + d] : 0.f;
-        if (c.mult == 1.f) v = xv;
-        if (c.y) v += c.post_w ? c.y[base + d] * post * (off + c.post_w[d]) : c.y[base + d];
-        if (c.y2) v += c.y2[base + d] * post2 * (off + c.post_w2[d]);
-        if (c.ff) v = fmaf(ff_gate, c.ff[base + d], v);
-        for (int k = 0; k < c.top; ++k)     // routed experts' results in choice order
-            v = fmaf(c.gate[(long long)m * c.top + k], c.expert_out[(long long)c.slot_of[(long long)m * c.top + k] * D + d], v);
-        if (c.bias) v += c.bias[d];
-        if (c.mult != 1.f) v = fmaf(c.mult, v, xv);
-        row[d] = v;
-        if (c.x_out) c.x_out[base + d] = v;
+#pragma unroll(V == 4 ? 1 : 4)
+    for (int d = first; d < D; d += step) {
+        float v[V], xv[V], t[V], w[V];
+#pragma unroll
+        for (int e = 0; e < V; ++e) xv[e] = 0.f;
+        if (c.x_in) loadv<V>(c.x_in + in_base + d, xv);
+#pragma unroll
+        for (int e = 0; e < V; ++e) v[e] = c.mult == 1.f ? xv[e] : 0.f;
+        if (c.y) {
+            loadv<V>(c.y + base + d, t);
+            if (c.post_w) {
+                loadv<V>(c.post_w + d, w);
+#pragma unroll
+                for (int e = 0; e < V; ++e) t[e] = t[e] * post * (off + w[e]);
+            }
+#pragma unroll
+            for (int e = 0; e < V; ++e) v[e] += t[e];
+        }
+        if (c.y2) {
+            loadv<V>(c.y2 + base + d, t);
+            loadv<V>(c.post_w2 + d, w);
+#pragma unroll
+            for (int e = 0; e < V; ++e) v[e] += t[e] * post2 * (off + w[e]);
+        }
+        if (c.ff) {
+            loadv<V>(c.ff + base + d, t);
+#pragma unroll
+            for (int e = 0; e < V; ++e) v[e] = fmaf(ff_gate, t[e], v[e]);
+        }
+        for (int k = 0; k < c.top; ++k) {   // routed experts' results in choice order
+            const float g = c.gate[(long long)m * c.top + k];
+            loadv<V>(c.expert_out + (long long)c.slot_of[(long long)m * c.top + k] * D + d, t);
+#pragma unroll
+            for (int e = 0; e < V; ++e) v[e] = fmaf(g, t[e], v[e]);
+        }
+        if (c.bias) {
+            loadv<V>(c.bias + d, t);
+#pragma unroll
+            for (int e = 0; e < V; ++e) v[e] += t[e];
+        }
+        if (c.mult != 1.f)
+#pragma unroll
+            for (int e = 0; e < V; ++e) v[e] = fmaf(c.mult, v[e], xv[e]);
+        storev<V>(row + d, v);
+        if (c.x_out) storev<V>(c.x_out + base + d, v);
     }
     if (c.next_w) {
         __syncthreads();
@@ -96,13 +160,23 @@ __global__ void row_close_kernel(RowClose c) {
             if (threadIdx.x == 0) gs[g] = 1.f / sqrtf(t / (float)Dg + c.eps);
         }
         __syncthreads();
-        for (int d = threadIdx.x; d < D; d += blockDim.x) {
-            float v = (row[d] - mean) * gs[d / Dg] * (off + c.next_w[d]);
-            if (c.next_b) v += c.next_b[d];
-            stx(c.hn, base + d, c.hn_f32, v);
-            if (c.hn_copy) c.hn_copy[base + d] = v;
+        for (int d = first; d < D; d += step) {
+            float v[V], w[V];
+            loadv<V>(row + d, v);
+            loadv<V>(c.next_w + d, w);
+            const float f = gs[d / Dg];      // V consecutive elements lie in one group
+#pragma unroll
+            for (int e = 0; e < V; ++e) v[e] = (v[e] - mean) * f * (off + w[e]);
+            if (c.next_b) {
+                loadv<V>(c.next_b + d, w);
+#pragma unroll
+                for (int e = 0; e < V; ++e) v[e] += w[e];
+            }
+            storevx<V>(c.hn, base + d, c.hn_f32, v);
+            if (c.hn_copy) storev<V>(c.hn_copy + base + d, v);
         }
     } else if (c.cat) {
+        __syncthreads();
         for (int d = threadIdx.x; d < D; d += blockDim.x) {
             stx(c.hn, 2 * base + d, c.hn_f32, row[d]);
             stx(c.hn, 2 * base + D + d, c.hn_f32, c.cat[base + d]);
@@ -232,8 +306,19 @@ int launch_row_close(const RowClose& c, cudaStream_t stream) {
     const size_t smem = (size_t)(c.D + 33 + MAX_NORM_GROUPS) * sizeof(float);
     if (smem > 200 * 1024) return set_error("row_close: width %d does not fit shared memory", c.D);
     static PerDeviceOnce once;
-    if (once.need()) ASD_CUDA(cudaFuncSetAttribute(row_close_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
-    row_close_kernel<<<c.M, row_threads(c.D), smem, stream>>>(c);
+    if (once.need()) {
+        ASD_CUDA(cudaFuncSetAttribute(row_close_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
+        ASD_CUDA(cudaFuncSetAttribute(row_close_kernel<4>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
+    }
+    uintptr_t at = 0;
+    for (const void* p : {(const void*)c.x_in, (const void*)c.y, (const void*)c.post_w, (const void*)c.bias, (const void*)c.x_out,
+                          (const void*)c.next_w, (const void*)c.hn, (const void*)c.expert_out, (const void*)c.y2,
+                          (const void*)c.post_w2, (const void*)c.ff, (const void*)c.next_b, (const void*)c.hn_copy})
+        at |= reinterpret_cast<uintptr_t>(p);
+    if (c.D % 4 == 0 && (c.D / c.groups) % 4 == 0 && (at & 15) == 0)
+        row_close_kernel<4><<<c.M, row_threads(c.D), smem, stream>>>(c);
+    else
+        row_close_kernel<1><<<c.M, row_threads(c.D), smem, stream>>>(c);
     count_launch(1);
     ASD_CUDA(cudaGetLastError());
     return 0;
