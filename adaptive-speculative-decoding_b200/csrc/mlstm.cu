@@ -76,17 +76,19 @@ __global__ void __launch_bounds__(MAXT, 1) mlstm_recurrence_kernel(MlstmArgs a) 
     float* st_slot = a.state + (size_t)slot * ring * entry;
     const size_t st_S = (size_t)head * dk * dv,
                  st_n = (size_t)H * dk * dv + ((size_t)head * gridDim.z + blockIdx.z) * (dk + 1), st_m = st_n + dk;
-    float S[ROWS];
+    float2 S[ROWS / 2];                   // rows in pairs: two of them per instruction
 #pragma unroll
-    for (int r = 0; r < ROWS; ++r) S[r] = 0.f;
+    for (int r = 0; r < ROWS / 2; ++r) S[r] = make_float2(0.f, 0.f);
     float n = 0.f, mrun = 0.f;            // lane r of a warp holds row r0 + r of the normaliser
     const bool n_ok = lane < ROWS && r0 + lane < dk;
     if (p0 > 0) {
         const float* src = st_slot + (size_t)((p0 - 1) % ring) * entry;
         if (col_ok) {
 #pragma unroll
-            for (int r = 0; r < ROWS; ++r)
-                if (r0 + r < dk) S[r] = src[st_S + (size_t)(r0 + r) * dv + col];
+            for (int r = 0; r < ROWS; r += 2) {
+                if (r0 + r < dk) S[r >> 1].x = src[st_S + (size_t)(r0 + r) * dv + col];
+                if (r0 + r + 1 < dk) S[r >> 1].y = src[st_S + (size_t)(r0 + r + 1) * dv + col];
+            }
         }
         if (n_ok) n = src[st_n + r0 + lane];
         mrun = src[st_m];
@@ -167,45 +169,49 @@ __global__ void __launch_bounds__(MAXT, 1) mlstm_recurrence_kernel(MlstmArgs a) 
             mrun = __shfl_sync(0xffffffffu, mlane, nt - 1);
             __syncwarp();
         }
-        for (int t = 0; t < nt; ++t) {
+        auto position = [&](int t) {
             const float keep = gates[t], put = gates[MAXC + t];
             const float4* k4 = reinterpret_cast<const float4*>(ks + t * dkp + r0);
             const float4* q4 = reinterpret_cast<const float4*>(qs + t * dkp + r0);
             const float pv = put * vs[t * 32 + lane];
-            float o0 = 0.f, o1 = 0.f;
+            const float2 keep2 = make_float2(keep, keep), pv2 = make_float2(pv, pv);
+            float2 oa = make_float2(0.f, 0.f), ob = make_float2(0.f, 0.f);
 #pragma unroll
             for (int r = 0; r < ROWS; r += 4) {
                 const float4 kk = k4[r >> 2], qq = q4[r >> 2];
-                S[r] = fmaf(kk.x, pv, keep * S[r]);
-                S[r + 1] = fmaf(kk.y, pv, keep * S[r + 1]);
-                S[r + 2] = fmaf(kk.z, pv, keep * S[r + 2]);
-                S[r + 3] = fmaf(kk.w, pv, keep * S[r + 3]);
-                o0 = fmaf(S[r], qq.x, o0);
-                o1 = fmaf(S[r + 1], qq.y, o1);
-                o0 = fmaf(S[r + 2], qq.z, o0);
-                o1 = fmaf(S[r + 3], qq.w, o1);
+                float2 &s0 = S[r >> 1], &s1 = S[(r >> 1) + 1];
+                s0 = fma2(make_float2(kk.x, kk.y), pv2, mul2(keep2, s0));
+                s1 = fma2(make_float2(kk.z, kk.w), pv2, mul2(keep2, s1));
+                oa = fma2(s0, make_float2(qq.x, qq.y), oa);
+                ob = fma2(s1, make_float2(qq.z, qq.w), ob);
             }
-            red[(t * RS + warp) * 32 + lane] = o0 + o1;
+            red[(t * RS + warp) * 32 + lane] = (oa.x + oa.y) + (ob.x + ob.y);
             float nq = 0.f;
             if (lane < ROWS) {
                 n = fmaf(ks[t * dkp + r0 + lane], put, keep * n);
                 nq = n * qs[t * dkp + r0 + lane];
             }
             redn[(t * RS + warp) * 32 + lane] = nq;
-            const int m = c0 + t;
-            if (t1 - m <= ring) {     // the last `ring` new positions leave their state behind
-                float* dst = st_slot + (size_t)((p0 + (m - t0)) % ring) * entry;
-                if (col_ok) {
+        };
+        const int plain = min(nt, max(0, t1 - ring - c0));      // positions that leave no state behind
+#pragma unroll 2
+        for (int t = 0; t < plain; ++t) position(t);
+        for (int t = plain; t < nt; ++t) {
+            position(t);
+            float* dst = st_slot + (size_t)((p0 + (c0 + t - t0)) % ring) * entry;
+            if (col_ok) {
 #pragma unroll
-                    for (int r = 0; r < ROWS; ++r)
-                        if (r0 + r < dk) dst[st_S + (size_t)(r0 + r) * dv + col] = S[r];
+                for (int r = 0; r < ROWS; r += 2) {
+                    if (r0 + r < dk) dst[st_S + (size_t)(r0 + r) * dv + col] = S[r >> 1].x;
+                    if (r0 + r + 1 < dk) dst[st_S + (size_t)(r0 + r + 1) * dv + col] = S[r >> 1].y;
                 }
-                if (n_ok) dst[st_n + r0 + lane] = n;
-                const float mt = __shfl_sync(0xffffffffu, mlane, t);
-                if (threadIdx.x == 0) dst[st_m] = mt;
             }
+            if (n_ok) dst[st_n + r0 + lane] = n;
+            const float mt = __shfl_sync(0xffffffffu, mlane, t);
+            if (threadIdx.x == 0) dst[st_m] = mt;
         }
         __syncthreads();   // the chunk's partial products are complete (and its buffer may be refilled)
+#pragma unroll 4
         for (int t = warp; t < nt; t += RS) {
             float nq = 0.f, o = 0.f;
             for (int w = 0; w < RS; ++w) {
@@ -331,7 +337,7 @@ int launch_mlstm_recurrence(const SeqIndex& ix, const int* cu_q, const int* seq_
     int ch = MAXC;   // positions per staged chunk; steps of few tokens stage (and clear) no more than they use
     while (ch > 1 && (long long)(ch / 2) * nseq >= ix.M) ch >>= 1;
     auto need = [&](int c) { return (size_t)total_floats(c, dkp, RS) * sizeof(float); };
-    while (ch > 1 && need(ch) > 96 * 1024) ch >>= 1;
+    while (ch > 1 && need(ch) > 112 * 1024) ch >>= 1;
     const size_t smem = need(ch);
     if (smem > 220 * 1024) return set_error("mlstm: key size %d does not fit shared memory", d.dk);
     dim3 grid(nseq, d.heads, (d.dv + 31) / 32);
