@@ -104,6 +104,21 @@ class DikopelConfigC(ctypes.Structure):
                 ("dtype", ctypes.c_int)]
 
 
+class NobonexLayerC(ctypes.Structure):
+    """mirror of ``asd_nobonex_layer_config``"""
+    _fields_ = [(n, ctypes.c_int) for n in (
+        "type", "kv_from", "heads", "kv_heads", "dim", "vdim", "conv", "rot_dims", "chunk", "state", "groups", "norm_groups",
+        "ff_kind", "ff", "experts", "top", "expert_ff")] + [(n, ctypes.c_float) for n in ("scale", "softcap", "limit")] + [
+        (n, ctypes.c_double) for n in ("rot_base", "yarn_factor", "yarn_original", "yarn_fast", "yarn_slow")]
+
+
+class NobonexConfigC(ctypes.Structure):
+    """mirror of ``asd_nobonex_config``"""
+    _fields_ = [("width", ctypes.c_int), ("vocab", ctypes.c_int), ("n_layers", ctypes.c_int), ("eps", ctypes.c_float),
+                ("embed_scale", ctypes.c_float), ("residual_mult", ctypes.c_float), ("max_tokens", ctypes.c_int),
+                ("page_size", ctypes.c_int), ("ring", ctypes.c_int), ("dtype", ctypes.c_int)]
+
+
 def library_path() -> str:
     return os.path.join(_HERE, "libasd_b200.so")
 
@@ -207,6 +222,16 @@ def lib() -> ctypes.CDLL:
         "asd_dikopel_forward": (i32, [vp, vp, vp, vp, i32, vp, vp, i32, i32, i32, vp, i32, vp, c.c_longlong, vp, vp]),
         "asd_dikopel_profile_read": (i32, [vp, vp, vp, i32]),
         "asd_dikopel_device_error": (i32, [vp]),
+        "asd_nobonex_create": (vp, [vp, vp]),
+        "asd_nobonex_destroy": (None, [vp]),
+        "asd_nobonex_set_tensor": (i32, [vp, i32, c.c_char_p, vp]),
+        "asd_nobonex_cache_bytes": (sz, [vp, i32]),
+        "asd_nobonex_state_bytes": (sz, [vp, i32]),
+        "asd_nobonex_set_cache": (i32, [vp, vp, i32, vp, i32, i32, vp]),
+        "asd_nobonex_set_option": (i32, [vp, c.c_char_p, i32]),
+        "asd_nobonex_forward": (i32, [vp, vp, vp, vp, i32, vp, vp, i32, i32, i32, vp, i32, vp, c.c_longlong, vp, vp]),
+        "asd_nobonex_profile_read": (i32, [vp, vp, vp, i32]),
+        "asd_nobonex_device_error": (i32, [vp]),
     }
     for name, (res, args) in sigs.items():
         fn = getattr(L, name, None)

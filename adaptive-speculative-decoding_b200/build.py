@@ -30,16 +30,18 @@ COMPONENTS = {
     "rivetar": ["rivetar_engine.cu", "gla.cu", "window_attention.cu"],
     "delta": ["delta_rule.cu"],                 # delta rules and short convolutions
     "mixattn": ["mixed_attention.cu", "mixed_attention_tc.cu", "sigmoid_attention.cu",
-                "sigmoid_attention_tc.cu"],
+                "decode_attention_tc.cu"],
     "mavipel": ["mavipel_engine.cu", "talking_attention.cu"],
     "lukopel": ["lukopel_engine.cu", "residual_streams.cu"],
     "dikopel": ["dikopel_engine.cu", "mlstm.cu"],
+    "nobonex": ["nobonex_engine.cu", "ssd.cu"],
     "qwen": ["engine.cu", "layers.cu", "attention.cu", "attention_tc.cu", "forward_persist.cu"],
     "sampling": ["api.cu", "sampler.cu", "stop_rule.cu"],
 }
 REQUIRES = {"mezilix": ("linear", "blocks", "latent", "rows"), "rivetar": ("linear", "blocks", "latent", "rows"),
             "mavipel": ("linear", "blocks", "rows", "delta"), "lukopel": ("linear", "blocks", "rows", "mixattn"),
-            "dikopel": ("linear", "blocks", "rows", "delta", "mixattn"), "qwen": ("linear",)}
+            "dikopel": ("linear", "blocks", "rows", "delta", "mixattn"),
+            "nobonex": ("linear", "blocks", "rows", "delta", "mixattn"), "qwen": ("linear",)}
 
 
 def all_components():

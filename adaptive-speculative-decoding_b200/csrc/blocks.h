@@ -153,6 +153,8 @@ struct MoeRouterInput {
     const float* correction = nullptr;   // [E]
     int groups = 1, keep = 1;
     float scale = 1.f;
+    int plain_scores = 0;          // sigmoid only: gate = s * scale, the chosen scores are not divided by their sum
+    float* slot_gate = nullptr;    // optional [M * top]: the gate of each slot (what multiplies an expert's INPUT row)
     int extra = 0;                 // w has `extra` more rows whose raw logits follow the experts' in logits_out [M][E + extra]
 };
 int launch_moe_route(const float* logits, const MoeRouterInput* in, int M, int E, int top, int* expert_of, float* gate,
@@ -208,6 +210,41 @@ struct RowClose {
     float* hn_copy = nullptr;           // [M][D]
 };
 int launch_row_close(const RowClose& c, cudaStream_t stream);
+// The close for layers whose norms are "dynamic tanh", N(x) = tanh(alpha * x) * w + b (alpha a device scalar; no mean, no
+// root mean square):  x_out = x_in + mult * post(y + sum of the token's expert results);  hn = next(x_out) in the engine's
+// element type.  Without y and experts x stays as it is (hn only); with `rows`, row r reads x_in[rows[r]].
+struct TanhNorm {
+    const float* w = nullptr;      // [D]
+    const float* b = nullptr;      // [D]
+    const float* alpha = nullptr;  // scalar
+};
+struct TanhClose {
+    const float* x_in = nullptr;   // [M][D]
+    const int* rows = nullptr;
+    const float* y = nullptr;      // [M][D]
+    const float* expert_out = nullptr;  // [M * top][D] rows by slot, added as they are
+    const int* slot_of = nullptr;       // [M][top]
+    int top = 0;
+    TanhNorm post;
+    float mult = 1.f;
+    float* x_out = nullptr;        // [M][D], may alias x_in
+    TanhNorm next;
+    void* hn = nullptr;
+    int hn_f32 = 0;
+    int M = 0, D = 0;
+};
+int launch_tanh_close(const TanhClose& c, cudaStream_t stream);
+// Gated feed-forward activations over rows of 2 F floats (gate half g, then up half u), out [rows][F] in the engine's
+// element type.  row_factor (optional, one per row) multiplies g and u first: for a layer without biases that is the same
+// as multiplying the layer's input row.
+enum { GATED_GELU_TANH = 0,   // gelu_tanh(g) * u
+       GATED_CLAMPED = 1 };   // c = min(g, limit): c * sigmoid(slope * c) * (clamp(u, -limit, limit) + 1)
+struct GatedAct {
+    int kind = GATED_GELU_TANH;
+    float limit = 0.f, slope = 1.702f;
+    const float* row_factor = nullptr;
+};
+int launch_gated_act(const float* z, void* out, int of32, long long rows, int F, const GatedAct& p, cudaStream_t stream);
 // x[m] = embed[token] with each of `groups` equal consecutive parts divided by its root mean square, times w; fp32
 int launch_embed_normed(const SeqIndex& ix, const void* embed, int wf32, const float* w, int groups, float eps, float* x,
                         int D, cudaStream_t stream);
@@ -293,11 +330,13 @@ int launch_lowrank_channels(const float* a, long long lda, const LowRankChannels
 // the last ring_n new positions of every sequence there and must follow the convolution.
 int launch_short_conv(const SeqIndex& ix, const float* in, long long ld, const float* taps, int n_taps, int C,
                       const float* ring, int ring_n, float* out, cudaStream_t stream);
-// The convolution and the commit in one call (a single launch for steps of one token per sequence).  residual = 0: as
-// above; 1: out[m][c] = in[m][c] + convolution, no activation.  out [M][C] in the engine's element type (of32).
+// The convolution and the commit in one call (a single launch for steps of one token per sequence).  CONV_SILU: as above;
+// CONV_RESIDUAL: out[m][c] = in[m][c] + convolution; CONV_PLAIN: the convolution alone; both without an activation.  bias
+// (optional [C]) is added to the convolution.  out [M][C] in the engine's element type (of32).
+enum { CONV_SILU = 0, CONV_RESIDUAL = 1, CONV_PLAIN = 2 };
 int launch_carried_conv(const SeqIndex& ix, const int* cu_q, int nseq, int max_qlen, const float* in, long long ld,
-                        const float* taps, int n_taps, int C, float* ring, int ring_n, int residual, void* out, int of32,
-                        cudaStream_t stream);
+                        const float* taps, int n_taps, int C, float* ring, int ring_n, int mode, void* out, int of32,
+                        cudaStream_t stream, const float* bias = nullptr);
 int launch_conv_commit(const SeqIndex& ix, const int* cu_q, int nseq, const float* in, long long ld, int C, float* ring,
                        int ring_n, cudaStream_t stream);
 // The vectors a position's recurrence step reads, rv fp32 [M][heads][3, 2 or 5][dk] and sc fp32 [M][heads][4] (layout in
@@ -332,12 +371,13 @@ int launch_delta_recurrence(const SeqIndex& ix, const int* cu_q, const int* seq_
                             float* state, int ring, float* out, cudaStream_t stream);
 // y[m][h][:] = o[m][h][:] / rms(o[m][h][:]) * w * gate[m][h][:] * scale, y = rows ldy apart in the engine's element
 // type.  w: [dv] shared by the heads or [heads * dv]; gate: fp32 rows ldg apart, taken as they are (gate_act 0), through a
-// sigmoid (1) or a silu (2).
+// sigmoid (1) or a silu (2).  gate_first: the gate multiplies before the root mean square is taken (o * gate is normed).
+// "Heads" may be any equal consecutive parts of a row.
 struct HeadNormGate {
     const float* gate = nullptr;
     long long ldg = 0;
     const float* w = nullptr;
-    int w_per_head = 0, gate_act = 0;
+    int w_per_head = 0, gate_act = 0, gate_first = 0;
     float eps = 0.f, scale = 1.f;
 };
 int launch_head_norm_gate(const float* o, const HeadNormGate& p, void* y, int of32, long long ldy, int M, int heads, int dv,
@@ -406,13 +446,18 @@ struct MixDims {
     // 1: the weight of a visible key is sigmoid(score + head_bias[head]), not normalised over the keys (no head mix then)
     int sigmoid = 0;
     const float* head_bias = nullptr;   // fp32 [heads], optional
+    float softcap = 0.f;                // > 0: scores are capped, softcap * tanh(score / softcap)
+    int gate_per_value = 0;             // 1: the gate has a value per result element ([heads * dv]) instead of one per head
 };
 // What the projections pass before the attention.  qkv fp32 rows (ld floats apart) = [heads * dk | kv_heads * dk |
 // kv_heads * dv].  Adds the biases (same layout, optional); RMS-norms queries and keys either head by head (weights [dk],
 // norm_whole = 0) or over the whole projection (weights [heads * dk] and [kv_heads * dk], norm_whole = 1); multiplies the
+// rotates the leading rot_dims coordinates of every query and key head by position * rot_freq[i], in pairs (2 i, 2 i + 1) or
+// (i, i + rot_dims / 2), cos and sin times rot_mag (after the norms; the angle is reduced to one turn in fp64); multiplies the
 // queries by 1 + temp_coef * ln(floor((position + 1) / temp_every) + 1) (temp_every 0: not) and by head_factor[head]
 // (optional); divides every value head by its root mean square (v_unit); leaves the queries in place and appends keys
-// and values to the cache.
+// and values to the cache.  v_from_k: rows are [heads * dk | kv_heads * dk] and the values are the keys before norm and
+// rotation (dv = dk).  q_only: rows hold queries alone and nothing is appended (a layer that reads another layer's cache).
 struct MixPost {
     const float* bias = nullptr;
     const float* q_norm = nullptr;
@@ -423,6 +468,10 @@ struct MixPost {
     const float* head_factor = nullptr;
     int v_unit = 0;
     float eps = 0.f;
+    const double* rot_freq = nullptr;   // fp64 [rot_dims / 2]
+    int rot_dims = 0, rot_interleaved = 0;
+    float rot_mag = 1.f;
+    int v_from_k = 0, q_only = 0;
 };
 int launch_mix_post(const SeqIndex& ix, float* qkv, long long ld, const MixDims& d, const MixPost& p,
                     const PagedRows& cache, cudaStream_t stream);
@@ -448,6 +497,31 @@ int launch_mix_attention(const SeqIndex& ix, const int* cu_q, const int* seq_slo
                          const float* q, long long ldq, const MixDims& d, const float* dist_bias, int far,
                          const float* talk, const float* gate, long long ldg, const PagedRows& cache, void* out, int of32,
                          long long ldo, const MixWork& ws, cudaStream_t stream);
+
+// ---------------------------------------------------------------------------------------------- ssd.cu
+// Scalar-decay state space recurrence (Mamba-2): per head a state S [dk][dv] in fp32 under one decay per position,
+//   dt = softplus(raw + dt_bias[head]);  S = exp(-exp(a_log[head]) dt) S + dt B x^T;  y = S^T C + skip[head] x,
+// with B and C (dk values each) shared by heads / groups heads.
+struct SsdDims {
+    int heads, groups, dk, dv;
+};
+struct SsdInput {
+    const float* x = nullptr;    // fp32 rows ld floats apart: heads * dv used
+    const float* b = nullptr;    // groups * dk used
+    const float* c = nullptr;
+    long long ld = 0;
+    const float* dt = nullptr;   // raw, fp32 rows ld_dt apart: one per head
+    long long ld_dt = 0;
+    const float* dt_bias = nullptr;   // [heads] each
+    const float* a_log = nullptr;
+    const float* skip = nullptr;
+};
+// state fp32 [slots][ring][heads][dk][dv]; entry position % ring holds the state after that position.  A sequence whose
+// first new position is 0 starts from zero, any other from entry (position - 1) % ring; the last `ring` new positions of
+// a sequence store theirs.  out fp32 [M][heads * dv].  mode 0: prompts run chunk by chunk on the tensor cores (fp32 operands
+// as two bf16 terms, fp32 state) where the sizes allow; 1: position by position in fp32.
+int launch_ssd_recurrence(const SeqIndex& ix, const int* cu_q, const int* seq_slot, int nseq, int max_qlen, const SsdInput& in,
+                          const SsdDims& d, float* state, int ring, float* out, int mode, cudaStream_t stream);
 
 // ---------------------------------------------------------------------------------------------- mlstm.cu
 // Matrix memory with exponential gates (mLSTM): per head a state S [dk][dv], a normaliser n [dk] and a running maximum M,

@@ -1,9 +1,11 @@
-// Steps of few tokens of the sigmoid attention on the tensor cores (bf16 cache rows; mma.sync m16n8k16, fp32 accumulation).
+// Steps of few tokens of attention with sigmoid or softmax weights on the tensor cores (bf16 cache rows; mma.sync m16n8k16, fp32 accumulation).
 // A CTA owns one sequence, one key/value group, up to sixteen (token, head) rows and one key share.  Its warps work on
 // 16-key tiles of their own, staged by cp.async in a ring per warp, so nothing but the end meets at a barrier: scores of the
-// sixteen rows against a tile, sigmoids in registers (they already stand in the layout of the next product's operand),
+// sixteen rows against a tile, weights in registers (they already stand in the layout of the next product's operand),
 // values.  Queries and weights enter as two bf16 terms each, so that scores and sums keep fp32 accuracy against the cache's
-// bf16 rows.  The weights are not normalised, so the warps' sums and the key shares simply add, in index order.
+// bf16 rows.  Sigmoid weights are not normalised, so the warps' sums and the key shares simply add, in index order.  Softmax:
+// every warp keeps a running maximum per row, against which its sums stand; the warps' sums are brought to their common
+// maximum at the end, and the key shares' sums by the merge.
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
 #include <math.h>
@@ -35,8 +37,10 @@ __host__ __device__ inline int smem_bytes(int dkp, int dvp, int NS) {
     return 2 * 16 * (dkp + 8) * 2 + (tiles > red ? tiles : red);
 }
 
-template <int NDV, int NS>
-__global__ void __launch_bounds__(NT) sigmoid_decode_tc_kernel(MixArgs a) {
+enum { D_SIGMOID = 0, D_SOFTMAX = 1, D_SOFTMAX_CAP = 2 };
+template <int NDV, int NS, int MODE>
+__global__ void __launch_bounds__(NT) decode_tc_kernel(MixArgs a) {
+    constexpr bool SOFT = MODE != D_SIGMOID;
     extern __shared__ __align__(16) unsigned char smraw[];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
     const int H = a.d.heads, G = a.d.kv_heads, rep = H / G, dk = a.d.dk, dv = a.d.dv, M = a.ix.M;
@@ -48,7 +52,9 @@ __global__ void __launch_bounds__(NT) sigmoid_decode_tc_kernel(MixArgs a) {
     if (nrows <= 0) return;
     const int p0 = a.ix.positions[q0], slot = a.seq_slot[b];
     const int last = p0 + (rb * 16 + nrows - 1) / rep;    // last position any row sees
-    const int ntile = last / KT + 1, per = (ntile + a.shares - 1) / a.shares;
+    // chunked mask: keys from the first row's chunk on
+    const int chunk = a.d.chunk, kmin = chunk > 0 ? (p0 + rb * 16 / rep) / chunk * chunk : 0;
+    const int ntile = (last - kmin) / KT + 1, per = (ntile + a.shares - 1) / a.shares;
     const int t0 = share * per, t1 = min(ntile, t0 + per);
     bf16* Qh = reinterpret_cast<bf16*>(smraw);
     bf16* Ql = Qh + 16 * DS;
@@ -73,12 +79,14 @@ __global__ void __launch_bounds__(NT) sigmoid_decode_tc_kernel(MixArgs a) {
             if (d >= dk) ring[s * tile_elems(dkp, DVP) + k * DS + d] = __float2bfloat16(0.f);
         }
 
-    int posr[2];
-    float hb[2];
+    int posr[2], lor[2];
+    float hb[2], mrun[2] = {-INFINITY, -INFINITY}, lrun[2] = {0.f, 0.f};
+    const float icap = MODE == D_SOFTMAX_CAP ? 1.f / a.d.softcap : 0.f;
 #pragma unroll
     for (int x = 0; x < 2; ++x) {
         const int r = g + 8 * x, gr = rb * 16 + r;
         posr[x] = r < nrows ? p0 + gr / rep : -1;
+        lor[x] = chunk > 0 ? posr[x] / chunk * chunk : 0;
         hb[x] = (r < nrows && a.d.head_bias) ? a.d.head_bias[c * rep + gr % rep] : 0.f;
     }
     float O[NDV][4];
@@ -90,7 +98,7 @@ __global__ void __launch_bounds__(NT) sigmoid_decode_tc_kernel(MixArgs a) {
 
     // tile of this warp's step i: t0 + warp + NW * i; the cache row of its key `lane` (lanes 0 - 15), -1 beyond the last key
     auto rows_of = [&](int i) {
-        const int t = t0 + warp + NW * i, j = t * KT + (lane & 15);
+        const int t = t0 + warp + NW * i, j = kmin + t * KT + (lane & 15);
         if (t >= t1 || j > last) return -1;
         return a.cache.page_table[(long long)slot * a.cache.max_pages + j / psz] * psz + j % psz;
     };
@@ -140,16 +148,55 @@ __global__ void __launch_bounds__(NT) sigmoid_decode_tc_kernel(MixArgs a) {
             mma_bf16(s[0], al, bq[0], bq[1]);
             mma_bf16(s[1], al, bq[2], bq[3]);
         }
-        const int j0 = (t0 + warp + NW * i) * KT;
+        const int j0 = kmin + (t0 + warp + NW * i) * KT;
         uint32_t ph[4], pl[4];
+        if (SOFT) {
+#pragma unroll
+            for (int x = 0; x < 2; ++x) {
+                float mx = -INFINITY;
+#pragma unroll
+                for (int n = 0; n < 2; ++n)
+#pragma unroll
+                    for (int e = 0; e < 2; ++e) {
+                        const int j = j0 + n * 8 + 2 * t4 + e;
+                        float v = s[n][2 * x + e] * a.d.scale;
+                        if (MODE == D_SOFTMAX_CAP) v = cap_score(v, a.d.softcap, icap);
+                        v = j <= posr[x] && j >= lor[x] ? v : -INFINITY;
+                        s[n][2 * x + e] = v;
+                        mx = fmaxf(mx, v);
+                    }
+                mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
+                mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
+                const float mnew = fmaxf(mrun[x], mx), ref = mnew > -INFINITY ? mnew : 0.f;
+                const float keep = expf(mrun[x] - ref);
+                float sum = 0.f;           // this thread's part of the row's sum; the quad's parts are added at the end
+#pragma unroll
+                for (int n = 0; n < 2; ++n)
+#pragma unroll
+                    for (int e = 0; e < 2; ++e) {
+                        s[n][2 * x + e] = expf(s[n][2 * x + e] - ref);
+                        sum += s[n][2 * x + e];
+                    }
+                lrun[x] = fmaf(lrun[x], keep, sum);
+                mrun[x] = mnew;
+                if (__any_sync(0xffffffffu, keep != 1.f))
+#pragma unroll
+                    for (int n = 0; n < NDV; ++n) O[n][2 * x] *= keep, O[n][2 * x + 1] *= keep;
+            }
+        }
 #pragma unroll
         for (int u = 0; u < 4; ++u) {
             const int x = u & 1, n = u >> 1;
             float w[2];
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
-                const float z = fmaf(s[n][2 * x + e], a.d.scale, hb[x]);
-                w[e] = j0 + n * 8 + 2 * t4 + e <= posr[x] ? __fdividef(1.f, 1.f + __expf(-z)) : 0.f;
+                if (SOFT) {
+                    w[e] = s[n][2 * x + e];
+                } else {
+                    const float z = fmaf(s[n][2 * x + e], a.d.scale, hb[x]);
+                    const int j = j0 + n * 8 + 2 * t4 + e;
+                    w[e] = j <= posr[x] && j >= lor[x] ? __fdividef(1.f, 1.f + __expf(-z)) : 0.f;
+                }
             }
             const bf16 h0 = __float2bfloat16(w[0]), h1 = __float2bfloat16(w[1]);
             ph[u] = (uint32_t)__bfloat16_as_ushort(h0) | ((uint32_t)__bfloat16_as_ushort(h1) << 16);
@@ -168,6 +215,14 @@ __global__ void __launch_bounds__(NT) sigmoid_decode_tc_kernel(MixArgs a) {
     cp_async_wait<0>();
     __syncthreads();          // every warp is done with its tiles: their place takes the sums
     float* red = reinterpret_cast<float*>(Ql + 16 * DS);
+    float* stat = reinterpret_cast<float*>(Qh);       // [NW][16] maxima, then sums, in the queries' place
+    if (SOFT)
+#pragma unroll
+        for (int x = 0; x < 2; ++x) {
+            lrun[x] += __shfl_xor_sync(0xffffffffu, lrun[x], 1);
+            lrun[x] += __shfl_xor_sync(0xffffffffu, lrun[x], 2);
+            if (t4 == 0) stat[warp * 16 + g + 8 * x] = mrun[x], stat[NW * 16 + warp * 16 + g + 8 * x] = lrun[x];
+        }
 #pragma unroll
     for (int n = 0; n < NDV; ++n)
 #pragma unroll
@@ -179,26 +234,50 @@ __global__ void __launch_bounds__(NT) sigmoid_decode_tc_kernel(MixArgs a) {
         const int r = idx / dv, col = idx - r * dv, gr = rb * 16 + r;
         const int m = q0 + gr / rep, h = c * rep + gr % rep;
         float v = 0.f;
+        if (SOFT) {
+            float mm = -INFINITY, l = 0.f;
 #pragma unroll
-        for (int w = 0; w < NW; ++w) v += red[((size_t)w * 16 + r) * DVP + col];
+            for (int w = 0; w < NW; ++w) mm = fmaxf(mm, stat[w * 16 + r]);
+#pragma unroll
+            for (int w = 0; w < NW; ++w) {
+                const float f = mm > -INFINITY ? expf(stat[w * 16 + r] - mm) : 0.f;
+                l = fmaf(f, stat[NW * 16 + w * 16 + r], l);
+                v = fmaf(f, red[((size_t)w * 16 + r) * DVP + col], v);
+            }
+            if (a.shares == 1) {
+                v = l > 0.f ? v / l : 0.f;
+            } else if (col == 0) {
+                a.stats[((long long)share * M + m) * H + h] = mm;
+                a.stats[((long long)(a.shares + share) * M + m) * H + h] = l;
+            }
+        } else {
+#pragma unroll
+            for (int w = 0; w < NW; ++w) v += red[((size_t)w * 16 + r) * DVP + col];
+        }
         if (a.shares == 1) {
-            const float gate = a.gate ? 1.f / (1.f + expf(-a.gate[(long long)m * a.ldg + h])) : 1.f;
-            stx(a.out, (long long)m * a.ldo + (long long)h * dv + col, a.of32, v * gate);
+            stx(a.out, (long long)m * a.ldo + (long long)h * dv + col, a.of32, v * mix_gate(a, m, h, col));
         } else {
             a.part[((long long)share * M + m) * H * dv + (long long)h * dv + col] = v;
         }
     }
 }
 
-template <int NDV, int NS>
-int launch_ns(const MixArgs& a, dim3 grid, size_t smem, cudaStream_t stream) {
+template <int NDV, int NS, int MODE>
+int launch_mode(const MixArgs& a, dim3 grid, size_t smem, cudaStream_t stream) {
+    auto kernel = decode_tc_kernel<NDV, NS, MODE>;
     static PerDeviceOnce once;
-    if (once.need())
-        ASD_CUDA(cudaFuncSetAttribute(sigmoid_decode_tc_kernel<NDV, NS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
-    sigmoid_decode_tc_kernel<NDV, NS><<<grid, NT, smem, stream>>>(a);
+    if (once.need()) ASD_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
+    kernel<<<grid, NT, smem, stream>>>(a);
     count_launch(1);
     ASD_CUDA(cudaGetLastError());
     return 0;
+}
+
+template <int NDV, int NS>
+int launch_ns(const MixArgs& a, dim3 grid, size_t smem, cudaStream_t stream) {
+    if (a.d.sigmoid) return launch_mode<NDV, NS, D_SIGMOID>(a, grid, smem, stream);
+    return a.d.softcap > 0.f ? launch_mode<NDV, NS, D_SOFTMAX_CAP>(a, grid, smem, stream)
+                             : launch_mode<NDV, NS, D_SOFTMAX>(a, grid, smem, stream);
 }
 
 template <int NDV>
@@ -212,21 +291,23 @@ int launch_ndv(const MixArgs& a, dim3 grid, cudaStream_t stream) {
 
 }  // namespace
 
-int launch_sigmoid_attention_decode_tc(MixArgs a, int nseq, int max_qlen, int max_kv_len, const MixWork& ws,
-                                       cudaStream_t stream) {
+int launch_attention_decode_tc(MixArgs a, int nseq, int max_qlen, int max_kv_len, const MixWork& ws, cudaStream_t stream) {
     const int H = a.d.heads, G = a.d.kv_heads, rep = H / G, M = a.ix.M, dk = a.d.dk, dv = a.d.dv;
-    if (a.cache.f32 || a.dist_bias || a.talk || a.d.chunk || dv > 256 || dk % 8 || dv % 8 || nseq > 65535) return 1;
+    if (a.cache.f32 || a.dist_bias || a.talk || (a.d.sigmoid && a.d.softcap > 0.f) || dv > 256 || dk % 8 || dv % 8 || nseq > 65535) return 1;
     if (reinterpret_cast<uintptr_t>(a.cache.pool) & 15) return 1;
     const int ndv = dv <= 32 ? 4 : (dv <= 64 ? 8 : (dv <= 96 ? 12 : (dv <= 128 ? 16 : 32)));
     a.dkp = (dk + 15) & ~15, a.dvp = ndv * 8;
     if (smem_bytes(a.dkp, a.dvp, 2) > 200 * 1024) return 1;
-    const int blocks = (max_qlen * rep + 15) / 16, ntile = (max_kv_len + KT - 1) / KT;
+    const int keys = a.d.chunk > 0 ? std::min(max_kv_len, a.d.chunk + max_qlen - 1) : max_kv_len;     // at most, of a block
+    const int blocks = (max_qlen * rep + 15) / 16, ntile = (keys + KT - 1) / KT;
     const long long base = (long long)nseq * G * blocks;
     if ((long long)G * blocks > 65535) return 1;
     // key shares: a few CTAs for each of the two places an SM has, four tiles per warp at least
     int shares = (int)std::min<long long>((888 + base - 1) / base, std::max(1, ntile / (4 * NW)));
     shares = std::max(1, std::min(shares, 64));
-    while (shares > 1 && (!ws.part || (long long)shares * M * H * dv > ws.part_elems)) --shares;
+    while (shares > 1 && (!ws.part || (long long)shares * M * H * dv > ws.part_elems ||
+                          (!a.d.sigmoid && (long long)2 * shares * M * H > ws.stats_elems)))
+        --shares;
     a.shares = shares;
     const dim3 grid(shares, nseq, G * blocks);
     const int rc = ndv == 4    ? launch_ndv<4>(a, grid, stream)
@@ -235,7 +316,7 @@ int launch_sigmoid_attention_decode_tc(MixArgs a, int nseq, int max_qlen, int ma
                    : ndv == 16 ? launch_ndv<16>(a, grid, stream)
                                : launch_ndv<32>(a, grid, stream);
     if (rc) return -1;
-    if (shares > 1 && launch_mix_merge(a, stream)) return -1;
+    if (shares > 1 && launch_mix_merge(a, stream, !a.d.sigmoid)) return -1;
     return 0;
 }
 

@@ -89,12 +89,13 @@ __global__ void __launch_bounds__(LC_CH) lowrank_channels_kernel(const float* a,
 // ------------------------------------------------------------------------------------------ short causal convolution
 // out[m][c] = silu( sum_j taps[c][j] * in[position - (n - 1 - j)][c] ): inputs of this forward come from the rows above
 // (a sequence's tokens are consecutive rows), earlier ones from the ring of carried inputs, zeros before position 0.
-// RESID: out = in + convolution, no activation, in the engine's element type.  SINGLE (one token per sequence): the thread
+// bias (optional [C]) is added to the sum.  MODE CONV_RESIDUAL: out = in + convolution; CONV_PLAIN: the convolution; neither
+// has an activation.  SINGLE (one token per sequence): the thread
 // that has read a channel's carried inputs stores its new one, which saves the commit launch; the entry it overwrites is
 // either the oldest input, read by this very thread, or older than any that is read.
-template <bool RESID, bool SINGLE>
+template <int MODE, bool SINGLE>
 __global__ void short_conv_kernel(SeqIndex ix, const float* in, long long ld, const float* taps, int n, int C,
-                                  const float* ring_in, float* ring, int ring_n, void* out, int of32) {
+                                  const float* ring_in, float* ring, int ring_n, void* out, int of32, const float* bias) {
     const int m = blockIdx.x;
     const int pos = ix.positions[m], slot = ix.token_slot[m];
     // how many rows above belong to the same sequence's preceding positions (at most n - 1 are needed)
@@ -125,7 +126,9 @@ __global__ void short_conv_kernel(SeqIndex ix, const float* in, long long ld, co
     for (int u = 0; u < 4; ++u) {
         const int c = cb + u * blockDim.x;
         if (c < C) {
-            stx(out, (long long)m * C + c, of32, RESID ? cur[u] + acc[u] : acc[u] / (1.f + expf(-acc[u])));
+            if (bias) acc[u] += __ldg(bias + c);
+            const float v = MODE == CONV_RESIDUAL ? cur[u] + acc[u] : (MODE == CONV_PLAIN ? acc[u] : acc[u] / (1.f + expf(-acc[u])));
+            stx(out, (long long)m * C + c, of32, v);
             if (SINGLE) ring[((long long)slot * ring_n + pos % ring_n) * C + c] = cur[u];
         }
     }
@@ -568,14 +571,47 @@ __global__ void head_norm_gate_kernel(const float* o, HeadNormGate p, void* y, i
     const float* src = o + (m * heads + h) * dv;
     const float* g = p.gate + m * p.ldg + (long long)h * dv;
     const float* w = p.w + (p.w_per_head ? (long long)h * dv : 0);
+    auto gate = [&](int i) {
+        const float gv = g[i];
+        return p.gate_act ? (p.gate_act == 2 ? gv : 1.f) * sigmoid_f(gv) : gv;
+    };
     float ss = 0.f;
-    for (int i = lane; i < dv; i += 32) ss = fmaf(src[i], src[i], ss);
+    for (int i = lane; i < dv; i += 32) {
+        const float v = p.gate_first ? src[i] * gate(i) : src[i];
+        ss = fmaf(v, v, ss);
+    }
     ss = warp_sum(ss);
     const float r = p.scale / sqrtf(ss / (float)dv + p.eps);
-    for (int i = lane; i < dv; i += 32) {
-        float gv = g[i];
-        if (p.gate_act) gv = (p.gate_act == 2 ? gv : 1.f) * sigmoid_f(gv);
-        stx(y, m * ldy + (long long)h * dv + i, of32, src[i] * r * w[i] * gv);
+    for (int i = lane; i < dv; i += 32) stx(y, m * ldy + (long long)h * dv + i, of32, src[i] * r * w[i] * gate(i));
+}
+
+// parts too long for a warp: a CTA each, its gated values kept in registers between the sum and the result
+constexpr int WIDE_T = 256, WIDE_V = 8;
+__global__ void __launch_bounds__(WIDE_T) part_norm_gate_kernel(const float* o, HeadNormGate p, void* y, int of32, long long ldy,
+                                                                int heads, int dv) {
+    __shared__ float red[33];
+    const int h = blockIdx.y;
+    const long long m = blockIdx.x;
+    const float* src = o + (m * heads + h) * dv;
+    const float* g = p.gate + m * p.ldg + (long long)h * dv;
+    const float* w = p.w + (p.w_per_head ? (long long)h * dv : 0);
+    float v[WIDE_V], gv[WIDE_V];
+    float ss = 0.f;
+#pragma unroll
+    for (int u = 0; u < WIDE_V; ++u) {
+        const int i = u * WIDE_T + threadIdx.x;
+        v[u] = gv[u] = 0.f;
+        if (i >= dv) continue;
+        v[u] = src[i], gv[u] = g[i];
+        if (p.gate_act) gv[u] = (p.gate_act == 2 ? gv[u] : 1.f) * sigmoid_f(gv[u]);
+        const float t = p.gate_first ? v[u] * gv[u] : v[u];
+        ss = fmaf(t, t, ss);
+    }
+    const float r = p.scale / sqrtf(block_sum(ss, red) / (float)dv + p.eps);
+#pragma unroll
+    for (int u = 0; u < WIDE_V; ++u) {
+        const int i = u * WIDE_T + threadIdx.x;
+        if (i < dv) stx(y, m * ldy + (long long)h * dv + i, of32, v[u] * r * w[i] * gv[u]);
     }
 }
 
@@ -612,16 +648,16 @@ int launch_short_conv(const SeqIndex& ix, const float* in, long long ld, const f
     const int threads = C >= 1024 ? 256 : 128;
     dim3 grid(ix.M, (C + 4 * threads - 1) / (4 * threads));
     if (grid.y > 65535) return set_error("short_conv: too many channels");
-    short_conv_kernel<false, false><<<grid, threads, 0, stream>>>(ix, in, ld, taps, n_taps, C, ring, nullptr,
-                                                                  ring_n > 0 ? ring_n : 1, out, 1);
+    short_conv_kernel<CONV_SILU, false><<<grid, threads, 0, stream>>>(ix, in, ld, taps, n_taps, C, ring, nullptr,
+                                                                      ring_n > 0 ? ring_n : 1, out, 1, nullptr);
     count_launch(1);
     ASD_CUDA(cudaGetLastError());
     return 0;
 }
 
 int launch_carried_conv(const SeqIndex& ix, const int* cu_q, int nseq, int max_qlen, const float* in, long long ld,
-                        const float* taps, int n_taps, int C, float* ring, int ring_n, int residual, void* out, int of32,
-                        cudaStream_t stream) {
+                        const float* taps, int n_taps, int C, float* ring, int ring_n, int mode, void* out, int of32,
+                        cudaStream_t stream, const float* bias) {
     if (ix.M <= 0 || C <= 0) return 0;
     if (short_conv_check(n_taps, ring, ring_n)) return -1;
     const bool single = max_qlen == 1 && ring_n > 0 && n_taps > 1;
@@ -629,14 +665,15 @@ int launch_carried_conv(const SeqIndex& ix, const int* cu_q, int nseq, int max_q
     dim3 grid(ix.M, (C + 4 * threads - 1) / (4 * threads));
     if (grid.y > 65535) return set_error("short_conv: too many channels");
     const int rn = ring_n > 0 ? ring_n : 1;
-    if (residual && single)
-        short_conv_kernel<true, true><<<grid, threads, 0, stream>>>(ix, in, ld, taps, n_taps, C, ring, ring, rn, out, of32);
-    else if (residual)
-        short_conv_kernel<true, false><<<grid, threads, 0, stream>>>(ix, in, ld, taps, n_taps, C, ring, nullptr, rn, out, of32);
-    else if (single)
-        short_conv_kernel<false, true><<<grid, threads, 0, stream>>>(ix, in, ld, taps, n_taps, C, ring, ring, rn, out, of32);
+    auto run = [&](auto kernel) {
+        kernel<<<grid, threads, 0, stream>>>(ix, in, ld, taps, n_taps, C, ring, single ? ring : nullptr, rn, out, of32, bias);
+    };
+    if (mode == CONV_RESIDUAL)
+        single ? run(short_conv_kernel<CONV_RESIDUAL, true>) : run(short_conv_kernel<CONV_RESIDUAL, false>);
+    else if (mode == CONV_PLAIN)
+        single ? run(short_conv_kernel<CONV_PLAIN, true>) : run(short_conv_kernel<CONV_PLAIN, false>);
     else
-        short_conv_kernel<false, false><<<grid, threads, 0, stream>>>(ix, in, ld, taps, n_taps, C, ring, nullptr, rn, out, of32);
+        single ? run(short_conv_kernel<CONV_SILU, true>) : run(short_conv_kernel<CONV_SILU, false>);
     count_launch(1);
     ASD_CUDA(cudaGetLastError());
     if (single || ring_n <= 0) return 0;
@@ -753,6 +790,12 @@ int launch_head_norm_gate(const float* o, const HeadNormGate& p, void* y, int of
                           cudaStream_t stream) {
     if (M <= 0) return 0;
     if (!p.w || !p.gate) return set_error("head_norm_gate: missing inputs");
+    if (dv > 512 && dv <= WIDE_T * WIDE_V && heads <= 65535) {
+        part_norm_gate_kernel<<<dim3(M, heads), WIDE_T, 0, stream>>>(o, p, y, of32, ldy, heads, dv);
+        count_launch(1);
+        ASD_CUDA(cudaGetLastError());
+        return 0;
+    }
     const int wpb = heads < 8 ? heads : 8;
     dim3 grid(M, (heads + wpb - 1) / wpb);
     head_norm_gate_kernel<<<grid, wpb * 32, 0, stream>>>(o, p, y, of32, ldy, heads, dv);

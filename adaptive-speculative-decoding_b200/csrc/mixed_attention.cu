@@ -233,6 +233,7 @@ __global__ void __launch_bounds__(NT) mix_attn_kernel(MixArgs a) {
                         const int jj = tx + 16 * y, j = kb + jj;
                         const bool ok = row_ok && i < nq && jj < nk && j <= pos && j >= lo;
                         float v = acc[x][y] * a.d.scale;
+                        if (a.d.softcap > 0.f) v = a.d.softcap * tanhf(v / a.d.softcap);
                         if (a.dist_bias && ok) v += a.dist_bias[(long long)min(pos - j, a.far) * H + h];
                         s[y] = ok ? v : -INFINITY;
                         tmax = fmaxf(tmax, s[y]);
@@ -342,8 +343,6 @@ __global__ void __launch_bounds__(NT) mix_attn_kernel(MixArgs a) {
         const int hh = rg / QT, i = rg % QT, h = c * rep + hh;
         if (i >= nq) continue;
         const int m = q_beg + i;
-        float gate = 1.f;
-        if (a.shares == 1 && a.gate) gate = 1.f / (1.f + expf(-a.gate[(long long)m * a.ldg + h]));
 #pragma unroll
         for (int cb = 0; cb < CB; ++cb)
 #pragma unroll
@@ -351,25 +350,40 @@ __global__ void __launch_bounds__(NT) mix_attn_kernel(MixArgs a) {
                 const int col = cb * 64 + tx * 4 + e;
                 if (col >= dv) continue;
                 if (a.shares == 1)
-                    stx(a.out, (long long)m * a.ldo + (long long)h * dv + col, a.of32, o[s][cb][e] * gate);
+                    stx(a.out, (long long)m * a.ldo + (long long)h * dv + col, a.of32, o[s][cb][e] * mix_gate(a, m, h, col));
                 else
                     a.part[((long long)share * M + m) * H * dv + (long long)h * dv + col] = o[s][cb][e];
             }
     }
 }
 
-// out[m][h][:] = sigmoid(gate[m][h]) * sum over the key shares (in index order) of their partial results
-__global__ void mix_merge_kernel(const float* part, int shares, int M, int H, int dv, const float* gate, long long ldg,
-                                 void* out, int of32, long long ldo) {
-    const int m = blockIdx.x, n = H * dv;
+// out[m][h][:] = sigmoid(gate) * sum over the key shares (in index order) of their partial results.  STATS: the shares hold
+// sums of exp(score - the share's maximum) times values; maxima and sums of exponentials stand in a.stats.
+template <bool STATS>
+__global__ void mix_merge_kernel(MixArgs a) {
+    const int m = blockIdx.x, M = a.ix.M, H = a.d.heads, dv = a.d.dv, n = H * dv, shares = a.shares;
     const int e = blockIdx.y * blockDim.x + threadIdx.x;
     if (e >= n) return;
-    float acc = 0.f;
-#pragma unroll 8
-    for (int s = 0; s < shares; ++s) acc += part[((long long)s * M + m) * n + e];
     const int h = e / dv;
-    if (gate) acc *= 1.f / (1.f + expf(-gate[(long long)m * ldg + h]));
-    stx(out, (long long)m * ldo + e, of32, acc);
+    float acc = 0.f;
+    if (STATS) {
+        const float* mx = a.stats + (long long)m * H + h;
+        const long long step = (long long)M * H;
+        float mm = -INFINITY, l = 0.f;
+#pragma unroll 8
+        for (int s = 0; s < shares; ++s) mm = fmaxf(mm, mx[s * step]);
+#pragma unroll 8
+        for (int s = 0; s < shares; ++s) {
+            const float ms = mx[s * step], w = ms > -INFINITY ? expf(ms - mm) : 0.f;
+            l = fmaf(w, mx[(shares + s) * step], l);
+            acc = fmaf(w, a.part[((long long)s * M + m) * n + e], acc);
+        }
+        acc = l > 0.f ? acc / l : 0.f;
+    } else {
+#pragma unroll 8
+        for (int s = 0; s < shares; ++s) acc += a.part[((long long)s * M + m) * n + e];
+    }
+    stx(a.out, (long long)m * a.ldo + e, a.of32, acc * mix_gate(a, m, h, e - h * dv));
 }
 
 // ---------------------------------------------------------------------------------------------- steps of few tokens
@@ -496,6 +510,7 @@ __global__ void __launch_bounds__(NT) mix_dec_scores_kernel(MixArgs a) {
                 if (l8 == 0 && live) {
                     const int h = c * rep + x;
                     v *= a.d.scale;
+                    if (a.d.softcap > 0.f) v = a.d.softcap * tanhf(v / a.d.softcap);
                     if (a.dist_bias) v += a.dist_bias[(long long)min(pos - (kmin + k0 + ki), a.far) * H + h];
                     srow[(long long)h * a.score_ld + k0 + ki] = v;
                 }
@@ -652,7 +667,7 @@ __global__ void __launch_bounds__(NT) mix_dec_apply_kernel(MixArgs a) {
 #pragma unroll
             for (int w = 0; w < NT / 32; ++w) v += red[((size_t)w * rep + x) * dvp + col];
             if (a.shares == 1) {
-                const float gate = a.gate ? 1.f / (1.f + expf(-a.gate[(long long)m * a.ldg + h])) : 1.f;
+                const float gate = mix_gate(a, m, h, col);
                 stx(a.out, (long long)m * a.ldo + (long long)h * dv + col, a.of32, v * gate);
             } else {
                 a.part[((long long)share * M + m) * H * dv + (long long)h * dv + col] = v;
@@ -661,62 +676,86 @@ __global__ void __launch_bounds__(NT) mix_dec_apply_kernel(MixArgs a) {
     }
 }
 
-// dynamic shared memory: the row (n floats) + per-head sums of squares and factors
+// A warp per query, key and value head in turn.  Dynamic shared memory: the row (n floats), the heads' sums of squares,
+// cos and sin of the token's angles.
 template <typename T>
 __global__ void mix_post_kernel(SeqIndex ix, float* qkv, long long ld, MixDims d, MixPost p, PagedRows cache) {
     extern __shared__ float sm[];
     const int H = d.heads, G = d.kv_heads, dk = d.dk, dv = d.dv;
-    const int nq = H * dk, nk = G * dk, nv = G * dv, n = nq + nk + nv, units = H + 2 * G;
+    const int nq = H * dk, nk = p.q_only ? 0 : G * dk, nv = p.q_only || p.v_from_k ? 0 : G * dv, n = nq + nk + nv;
+    const int ku = H + (p.q_only ? 0 : G), units = ku + (nv ? G : 0);      // query heads, key heads, value heads
     float* row = sm;
-    float* fac = sm + n;
-    const int m = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, nw = blockDim.x >> 5;
+    float* ss_of = sm + n;
+    float* cs = ss_of + H + 2 * G;
+    const int m = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
     float* src = qkv + (long long)m * ld;
-    for (int i = tid; i < n; i += blockDim.x) row[i] = src[i] + (p.bias ? p.bias[i] : 0.f);
-    __syncthreads();
-    // sum of squares of every query head, key head and value head
+    const int pos = ix.positions[m], half = p.rot_dims >> 1;
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+        constexpr double TURN = 6.283185307179586476925;
+        const double ang = (double)pos * p.rot_freq[i];
+        float sn, c;
+        sincosf((float)(ang - TURN * rint(ang / TURN)), &sn, &c);
+        cs[i] = c * p.rot_mag, cs[half + i] = sn * p.rot_mag;
+    }
     for (int u = warp; u < units; u += nw) {
-        const int beg = u < H ? u * dk : (u < H + G ? nq + (u - H) * dk : nq + nk + (u - H - G) * dv);
-        const int len = u < H + G ? dk : dv;
+        const int beg = u < ku ? u * dk : nq + nk + (u - ku) * dv, len = u < ku ? dk : dv;
         float ss = 0.f;
-        for (int i = lane; i < len; i += 32) ss += row[beg + i] * row[beg + i];
+        for (int i = lane; i < len; i += 32) {
+            const float v = src[beg + i] + (p.bias ? p.bias[beg + i] : 0.f);
+            row[beg + i] = v;
+            ss = fmaf(v, v, ss);
+        }
         ss = warp_sum(ss);
-        if (lane == 0) fac[u] = ss;
+        if (lane == 0) ss_of[u] = ss;
     }
     __syncthreads();
-    if (tid == 0) {
-        const int pos = ix.positions[m];
-        const float temp = p.temp_every > 0 ? 1.f + p.temp_coef * logf((float)((pos + 1) / p.temp_every) + 1.f) : 1.f;
-        float wq = 0.f, wk = 0.f;
-        if (p.norm_whole) {
-            for (int u = 0; u < H; ++u) wq += fac[u];
-            for (int u = 0; u < G; ++u) wk += fac[H + u];
-            wq = 1.f / sqrtf(wq / (float)nq + p.eps), wk = 1.f / sqrtf(wk / (float)nk + p.eps);
+    float wq = 0.f, wk = 0.f;          // norms over whole projections
+    if (p.norm_whole) {
+        for (int u = lane; u < H; u += 32) wq += ss_of[u];
+        wq = 1.f / sqrtf(warp_sum(wq) / (float)nq + p.eps);
+        if (nk) {
+            for (int u = H + lane; u < H + G; u += 32) wk += ss_of[u];
+            wk = 1.f / sqrtf(warp_sum(wk) / (float)nk + p.eps);
         }
-        for (int u = 0; u < H; ++u) {
-            float f = !p.q_norm ? 1.f : (p.norm_whole ? wq : 1.f / sqrtf(fac[u] / (float)dk + p.eps));
+    }
+    const float temp = p.temp_every > 0 ? 1.f + p.temp_coef * logf((float)((pos + 1) / p.temp_every) + 1.f) : 1.f;
+    const int slot = ix.token_slot[m];
+    T* dst = nullptr;
+    if (!p.q_only) {
+        const int page = cache.page_table[(long long)slot * cache.max_pages + pos / cache.page_size];
+        dst = static_cast<T*>(cache.pool) + ((long long)page * cache.page_size + pos % cache.page_size) * (G * (dk + dv));
+    }
+    for (int u = warp; u < units; u += nw) {
+        if (u >= ku) {                                     // a value head
+            const int g = u - ku;
+            const float f = p.v_unit ? 1.f / sqrtf(ss_of[u] / (float)dv + p.eps) : 1.f;
+            for (int i = lane; i < dv; i += 32) stf(dst + G * dk + g * dv + i, row[nq + nk + g * dv + i] * f);
+            continue;
+        }
+        const bool is_q = u < H;
+        const float* nw_ = is_q ? p.q_norm : p.k_norm;
+        float f = 1.f;
+        if (nw_) f = p.norm_whole ? (is_q ? wq : wk) : 1.f / sqrtf(ss_of[u] / (float)dk + p.eps);
+        if (is_q) {
             f *= temp;
             if (p.head_factor) f *= p.head_factor[u];
-            fac[u] = f;
         }
-        for (int u = 0; u < G; ++u)
-            fac[H + u] = !p.k_norm ? 1.f : (p.norm_whole ? wk : 1.f / sqrtf(fac[H + u] / (float)dk + p.eps));
-        for (int u = 0; u < G; ++u) fac[H + G + u] = p.v_unit ? 1.f / sqrtf(fac[H + G + u] / (float)dv + p.eps) : 1.f;
-    }
-    __syncthreads();
-    const int pos = ix.positions[m], slot = ix.token_slot[m];
-    const int page = cache.page_table[(long long)slot * cache.max_pages + pos / cache.page_size];
-    T* dst = static_cast<T*>(cache.pool) + ((long long)page * cache.page_size + pos % cache.page_size) * (nk + nv);
-    for (int i = tid; i < n; i += blockDim.x) {
-        if (i < nq) {
-            const float w = p.q_norm ? p.q_norm[p.norm_whole ? i : i % dk] : 1.f;
-            src[i] = row[i] * fac[i / dk] * w;
-        } else if (i < nq + nk) {
-            const int e = i - nq;
-            const float w = p.k_norm ? p.k_norm[p.norm_whole ? e : e % dk] : 1.f;
-            stf(dst + e, row[i] * fac[H + e / dk] * w);
-        } else {
-            const int e = i - nq - nk;
-            stf(dst + nk + e, row[i] * fac[H + G + e / dv]);
+        const float* r = row + u * dk;
+        const float* w = nw_ ? nw_ + (p.norm_whole ? (is_q ? u : u - H) * dk : 0) : nullptr;
+        for (int i = lane; i < dk; i += 32) {
+            float v = r[i] * f * (w ? w[i] : 1.f);
+            if (i < p.rot_dims) {
+                const int j = p.rot_interleaved ? i ^ 1 : (i < half ? i + half : i - half);
+                const int pair = p.rot_interleaved ? i >> 1 : (i < half ? i : j);
+                const float o = r[j] * f * (w ? w[j] : 1.f);
+                v = fmaf(v, cs[pair], i < j ? -o * cs[half + pair] : o * cs[half + pair]);
+            }
+            if (is_q) {
+                src[u * dk + i] = v;
+            } else {
+                stf(dst + (u - H) * dk + i, v);
+                if (p.v_from_k) stf(dst + G * dk + (u - H) * dv + i, r[i] * (p.v_unit ? 1.f / sqrtf(ss_of[u] / (float)dk + p.eps) : 1.f));
+            }
         }
     }
 }
@@ -737,7 +776,10 @@ __global__ void mix_append_kernel(SeqIndex ix, const float* qkv, long long ld, i
 int launch_mix_post(const SeqIndex& ix, float* qkv, long long ld, const MixDims& d, const MixPost& p,
                     const PagedRows& cache, cudaStream_t stream) {
     if (ix.M <= 0) return 0;
-    if (!p.bias && !p.q_norm && !p.k_norm && !p.temp_every && !p.head_factor && !p.v_unit) {
+    if (p.v_from_k && (p.q_only || d.dv != d.dk)) return set_error("mix_post: values from keys of another size");
+    if (p.rot_dims > 0 && (!p.rot_freq || p.rot_dims % 2 || p.rot_dims > d.dk)) return set_error("mix_post: bad rotation");
+    if (!p.bias && !p.q_norm && !p.k_norm && !p.temp_every && !p.head_factor && !p.v_unit && !p.rot_dims && !p.v_from_k) {
+        if (p.q_only) return 0;
         const int nq = d.heads * d.dk, nkv = d.kv_heads * (d.dk + d.dv), threads = nkv >= 1024 ? 256 : 128;
         if (cache.f32)
             mix_append_kernel<float><<<ix.M, threads, 0, stream>>>(ix, qkv, ld, nq, nkv, cache);
@@ -747,8 +789,9 @@ int launch_mix_post(const SeqIndex& ix, float* qkv, long long ld, const MixDims&
         ASD_CUDA(cudaGetLastError());
         return 0;
     }
-    const int n = d.heads * d.dk + d.kv_heads * (d.dk + d.dv), units = d.heads + 2 * d.kv_heads;
-    const size_t smem = (size_t)(n + units) * sizeof(float);
+    const int n = d.heads * d.dk + (p.q_only ? 0 : d.kv_heads * (d.dk + (p.v_from_k ? 0 : d.dv)));
+    const size_t smem = (size_t)(n + d.heads + 2 * d.kv_heads + p.rot_dims) * sizeof(float);
+    const int threads = n >= 2048 ? 256 : 128;
     if (smem > 200 * 1024) return set_error("mix_post: a row of %d values does not fit shared memory", n);
     static PerDeviceOnce once;
     if (once.need()) {
@@ -756,17 +799,20 @@ int launch_mix_post(const SeqIndex& ix, float* qkv, long long ld, const MixDims&
         ASD_CUDA(cudaFuncSetAttribute(mix_post_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
     }
     if (cache.f32)
-        mix_post_kernel<float><<<ix.M, 128, smem, stream>>>(ix, qkv, ld, d, p, cache);
+        mix_post_kernel<float><<<ix.M, threads, smem, stream>>>(ix, qkv, ld, d, p, cache);
     else
-        mix_post_kernel<__nv_bfloat16><<<ix.M, 128, smem, stream>>>(ix, qkv, ld, d, p, cache);
+        mix_post_kernel<__nv_bfloat16><<<ix.M, threads, smem, stream>>>(ix, qkv, ld, d, p, cache);
     count_launch(1);
     ASD_CUDA(cudaGetLastError());
     return 0;
 }
 
-int launch_mix_merge(const MixArgs& a, cudaStream_t stream) {
+int launch_mix_merge(const MixArgs& a, cudaStream_t stream, bool stats) {
     const dim3 grid(a.ix.M, (a.d.heads * a.d.dv + 255) / 256);
-    mix_merge_kernel<<<grid, 256, 0, stream>>>(a.part, a.shares, a.ix.M, a.d.heads, a.d.dv, a.gate, a.ldg, a.out, a.of32, a.ldo);
+    if (stats)
+        mix_merge_kernel<true><<<grid, 256, 0, stream>>>(a);
+    else
+        mix_merge_kernel<false><<<grid, 256, 0, stream>>>(a);
     count_launch(1);
     ASD_CUDA(cudaGetLastError());
     return 0;
@@ -857,8 +903,8 @@ int launch_mix_attention(const SeqIndex& ix, const int* cu_q, const int* seq_slo
     a.QT = 1, a.shares = 1, a.gp = 1, a.rag = 1;
     a.vec = (d.dk % 4 == 0 && d.dv % 4 == 0) ? 1 : 0;
     // steps of few tokens; prompts of a bf16 engine on the tensor cores; else (and for sizes those refuse) the CUDA cores
-    if (d.sigmoid && max_qlen < 8 && ws.mode == 0) {
-        const int rc = launch_sigmoid_attention_decode_tc(a, nseq, max_qlen, max_kv_len, ws, stream);
+    if (max_qlen < 8 && ws.mode == 0) {
+        const int rc = launch_attention_decode_tc(a, nseq, max_qlen, max_kv_len, ws, stream);
         if (rc <= 0) return rc;
     }
     if (max_qlen <= 4 && ws.mode != 1) {

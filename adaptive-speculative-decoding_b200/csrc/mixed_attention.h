@@ -4,6 +4,7 @@
 #include <cuda_runtime.h>
 
 #include "blocks.h"
+#include "elem.cuh"
 
 namespace asd {
 
@@ -30,6 +31,21 @@ struct MixArgs {
     int QT, shares, gp, rag, dkp, dvp, vec;
 };
 
+// sigmoid of the gate of one result element (1 without a gate)
+__device__ __forceinline__ float mix_gate(const MixArgs& a, long long m, int h, int col) {
+    if (!a.gate) return 1.f;
+    return 1.f / (1.f + expf(-a.gate[m * a.ldg + (a.d.gate_per_value ? h * a.d.dv + col : h)]));
+}
+
+// cap * tanh(v / cap): the Taylor series of tanh to the seventh power below 1/4, 1 - 2 / (1 + e^(2a)) above; relative error
+// below 1e-6
+__device__ __forceinline__ float cap_score(float v, float cap, float icap) {
+    const float a = fabsf(v) * icap, a2 = a * a;
+    const float big = 1.f - __fdividef(2.f, 1.f + __expf(2.f * a));
+    const float small = a * fmaf(a2, fmaf(a2, fmaf(a2, -17.f / 315.f, 2.f / 15.f), -1.f / 3.f), 1.f);
+    return copysignf(cap * (a < 0.25f ? small : big), v);
+}
+
 // Prompts and portions of a bf16 engine on the tensor cores (mma.sync, fp32 operands as two bf16 terms).  Returns 1 if
 // these sizes are not taken (the caller then runs the CUDA-core kernels), 0 after the launches, -1 on an error.
 int launch_mix_attention_tc(MixArgs a, int nseq, int max_qlen, int max_kv_len, const MixWork& ws, cudaStream_t stream);
@@ -37,10 +53,11 @@ int launch_mix_attention_tc(MixArgs a, int nseq, int max_qlen, int max_kv_len, c
 int launch_mix_attention_decode(MixArgs a, int nseq, int max_kv_len, const MixWork& ws, cudaStream_t stream);
 // The same with sigmoid weights (sigmoid_attention.cu): one pass.  Same returns.
 int launch_sigmoid_attention_decode(MixArgs a, int max_kv_len, const MixWork& ws, cudaStream_t stream);
-// And on the tensor cores for bf16 cache rows (sigmoid_attention_tc.cu).  Same returns.
-int launch_sigmoid_attention_decode_tc(MixArgs a, int nseq, int max_qlen, int max_kv_len, const MixWork& ws,
+// Steps of few tokens on the tensor cores for bf16 cache rows, sigmoid or softmax weights without a head mix or distance bias
+// (decode_attention_tc.cu).  Same returns.
+int launch_attention_decode_tc(MixArgs a, int nseq, int max_qlen, int max_kv_len, const MixWork& ws,
                                        cudaStream_t stream);
 // sums the key shares' partial results in index order, applies the gates, writes the engine's element type
-int launch_mix_merge(const MixArgs& a, cudaStream_t stream);
+int launch_mix_merge(const MixArgs& a, cudaStream_t stream, bool stats = false);
 
 }  // namespace asd

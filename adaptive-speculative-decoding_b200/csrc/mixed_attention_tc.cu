@@ -78,7 +78,7 @@ __device__ __forceinline__ void stage_rows(const bf16* pool, const long long* ro
 // one share): no first pass at all; the running maximum rescales the sums tile by tile and the division by the softmax sum
 // comes last.  SIGMOID: the weights are sigmoids and need no statistics.
 enum { TWO_PASS = 0, ONLINE = 1, SIGMOID = 2 };
-template <int KT, int NDV, bool APPLY, bool TALK, int MODE>
+template <int KT, int NDV, bool APPLY, bool TALK, int MODE, bool CAP>
 __global__ void __launch_bounds__(NT) mix_tc_kernel(MixArgs a) {
     constexpr bool ONE = MODE == ONLINE;
     extern __shared__ __align__(16) unsigned char smraw[];
@@ -107,6 +107,7 @@ __global__ void __launch_bounds__(NT) mix_tc_kernel(MixArgs a) {
     float* Lr = reinterpret_cast<float*>(smraw + L.l);
     long long* rowoff = reinterpret_cast<long long*>(smraw + L.off);
     const int M = a.ix.M;
+    const float icap = CAP ? 1.f / a.d.softcap : 0.f;
     const int p0 = a.ix.positions[q_beg], p1 = p0 + nq - 1;
     const int kmin = chunk > 0 ? (p0 / chunk) * chunk : 0;
     const int ntile = (p1 - kmin) / KT + 1;
@@ -247,6 +248,7 @@ __global__ void __launch_bounds__(NT) mix_tc_kernel(MixArgs a) {
                     const int x = e >> 1, col = n * 8 + 2 * t + (e & 1), j = kb + col;
                     const bool ok = okx[x] && col < nk && j <= posx[x] && j >= lox[x];
                     float v = s[n][e] * a.d.scale;
+                    if (CAP) v = cap_score(v, a.d.softcap, icap);
                     if (a.dist_bias && ok) v += a.dist_bias[(long long)min(posx[x] - j, a.far) * H + hx[x]];
                     if (MODE == SIGMOID) {
                         s[n][e] = ok ? __fdividef(1.f, 1.f + __expf(-(v + hbx[x]))) : 0.f;
@@ -400,8 +402,6 @@ __global__ void __launch_bounds__(NT) mix_tc_kernel(MixArgs a) {
     for (int x = 0; x < 2; ++x) {
         if (!okx[x]) continue;
         const int m = q_beg + ix_[x], h = hx[x];
-        float gate = 1.f;
-        if (a.shares == 1 && a.gate) gate = 1.f / (1.f + expf(-a.gate[(long long)m * a.ldg + h]));
 #pragma unroll
         for (int n = 0; n < NDV; ++n)
 #pragma unroll
@@ -410,20 +410,19 @@ __global__ void __launch_bounds__(NT) mix_tc_kernel(MixArgs a) {
                 if (col >= dv) continue;
                 const float v = O[n][2 * x + e];
                 if (a.shares == 1)
-                    stx(a.out, (long long)m * a.ldo + (long long)h * dv + col, a.of32, v * gate);
+                    stx(a.out, (long long)m * a.ldo + (long long)h * dv + col, a.of32, v * mix_gate(a, m, h, col));
                 else
                     a.part[((long long)share * M + m) * H * dv + (long long)h * dv + col] = v;
             }
     }
 }
 
-template <int KT, int NDV, bool APPLY, bool TALK, int MODE>
+template <int KT, int NDV, bool APPLY, bool TALK, int MODE, bool CAP = false>
 int launch_tc(const MixArgs& a, dim3 grid, size_t smem, cudaStream_t stream) {
+    auto kernel = mix_tc_kernel<KT, NDV, APPLY, TALK, MODE, CAP>;
     static PerDeviceOnce once;
-    if (once.need())
-        ASD_CUDA(cudaFuncSetAttribute(mix_tc_kernel<KT, NDV, APPLY, TALK, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                      220 * 1024));
-    mix_tc_kernel<KT, NDV, APPLY, TALK, MODE><<<grid, NT, smem, stream>>>(a);
+    if (once.need()) ASD_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
+    kernel<<<grid, NT, smem, stream>>>(a);
     count_launch(1);
     ASD_CUDA(cudaGetLastError());
     return 0;
@@ -433,13 +432,18 @@ template <int KT, int NDV>
 int launch_apply(const MixArgs& a, int mode, dim3 grid, size_t smem, cudaStream_t stream) {
     if (a.talk) return launch_tc<KT, NDV, true, true, TWO_PASS>(a, grid, smem, stream);
     if (mode == SIGMOID) return launch_tc<KT, NDV, true, false, SIGMOID>(a, grid, smem, stream);
+    if (a.d.softcap > 0.f)
+        return mode == ONLINE ? launch_tc<KT, NDV, true, false, ONLINE, true>(a, grid, smem, stream)
+                              : launch_tc<KT, NDV, true, false, TWO_PASS, true>(a, grid, smem, stream);
     return mode == ONLINE ? launch_tc<KT, NDV, true, false, ONLINE>(a, grid, smem, stream)
                           : launch_tc<KT, NDV, true, false, TWO_PASS>(a, grid, smem, stream);
 }
 
 template <int KT>
 int launch_passes(const MixArgs& a, int mode, int ndv, dim3 grid, size_t smem_stats, size_t smem_apply, cudaStream_t stream) {
-    if (mode == TWO_PASS && launch_tc<KT, 4, false, false, TWO_PASS>(a, grid, smem_stats, stream)) return -1;
+    if (mode == TWO_PASS && (a.d.softcap > 0.f ? launch_tc<KT, 4, false, false, TWO_PASS, true>(a, grid, smem_stats, stream)
+                                               : launch_tc<KT, 4, false, false, TWO_PASS>(a, grid, smem_stats, stream)))
+        return -1;
     return ndv == 4 ? launch_apply<KT, 4>(a, mode, grid, smem_apply, stream)
                     : (ndv == 8 ? launch_apply<KT, 8>(a, mode, grid, smem_apply, stream)
                                 : launch_apply<KT, 16>(a, mode, grid, smem_apply, stream));
@@ -451,6 +455,7 @@ int launch_mix_attention_tc(MixArgs a, int nseq, int max_qlen, int max_kv_len, c
     const int H = a.d.heads, G = a.d.kv_heads, rep = H / G, dk = a.d.dk, dv = a.d.dv;
     if (a.cache.f32 || dv > 128 || max_qlen < 8 || (reinterpret_cast<uintptr_t>(a.cache.pool) & 15)) return 1;
     const bool talk = a.talk != nullptr;
+    if (a.d.softcap > 0.f && (talk || a.d.sigmoid)) return 1;      // capped scores: plain softmax only
     const int ndv = dv <= 32 ? 4 : (dv <= 64 ? 8 : 16);
     const int dkp = (dk + 15) & ~15, DS = dkp + 8, VS = ndv * 8 + 8;
     // queries per tile and key/value groups per CTA: rows = groups * rep * QT <= 128, a multiple of 16, and every block of

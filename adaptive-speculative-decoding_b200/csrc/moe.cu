@@ -18,6 +18,8 @@ struct RouteChoice {
     int top, renorm, sigmoid, groups, keep;
     const float* correction;
     float scale;
+    int plain;             // sigmoid scores are the gates as they are
+    float* slot_gate;      // optional [M * top]: the gate of each slot
 };
 
 // One warp chooses a token's experts from its logits z[E] and writes their indices and gates; counts take one each.
@@ -98,7 +100,7 @@ __device__ void choose_experts(const float* z, int E, const RouteChoice& c, floa
         __syncwarp();
     }
     if (lane == 0 && c.sigmoid) {
-        const float r = c.scale / (chosen + 1e-20f);
+        const float r = c.plain ? c.scale : c.scale / (chosen + 1e-20f);
         for (int k = 0; k < c.top; ++k) gate[k] *= r;
     } else if (lane == 0 && c.renorm) {   // gates over the chosen alone: e^(z - max) / sum of the chosen e^(z - max)
         const float r = 1.f / (chosen * inv);
@@ -182,6 +184,7 @@ __global__ void __launch_bounds__(256) moe_route_small_kernel(const float* logit
         const int slot = off[e] + atomicAdd(&cnt[e], 1);
         sorted_tok[slot] = i / top;
         slot_of[i] = slot;
+        if (c.slot_gate) c.slot_gate[slot] = gate[i];
     }
 }
 
@@ -255,13 +258,14 @@ __global__ void moe_offsets_kernel(int* counters, int* group_off, int E) {
 }
 
 __global__ void moe_scatter_kernel(const int* expert_of, int n, int top, int E, const int* group_off, int* counters,
-                                   int* sorted_tok, int* slot_of) {
+                                   int* sorted_tok, int* slot_of, const float* gate, float* slot_gate) {
     const int i = blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= n) return;
     const int e = expert_of[i];
     const int slot = group_off[e] + atomicAdd(&counters[E + e], 1);
     sorted_tok[slot] = i / top;
     slot_of[i] = slot;
+    if (slot_gate) slot_gate[slot] = gate[i];
 }
 
 template <int NJ, int NTOK>
@@ -294,8 +298,9 @@ int launch_moe_route(const float* logits, const MoeRouterInput* in, int M, int E
     if (E <= 0 || top <= 0 || top > E) return set_error("moe: need 0 < top <= experts (top %d, experts %d)", top, E);
     if ((size_t)E * 8 * sizeof(float) > 48 * 1024) return set_error("moe: more than 1536 experts");
     if (!logits && !in) return set_error("moe: neither logits nor router inputs");
-    RouteChoice c{top, 0, 0, 1, 1, nullptr, 1.f};
-    if (in) c = RouteChoice{top, in->renorm, in->sigmoid, in->groups, in->keep, in->correction, in->scale};
+    RouteChoice c{top, 0, 0, 1, 1, nullptr, 1.f, 0, nullptr};
+    if (in)
+        c = RouteChoice{top, in->renorm, in->sigmoid, in->groups, in->keep, in->correction, in->scale, in->plain_scores, in->slot_gate};
     if (c.sigmoid) {
         if (!in->logits_out) return set_error("moe: sigmoid scores need logits_out");
         if (c.groups < 1 || E % c.groups || c.keep < 1 || c.keep > c.groups || top > c.keep * (E / c.groups))
@@ -323,7 +328,8 @@ int launch_moe_route(const float* logits, const MoeRouterInput* in, int M, int E
         nullptr, M, E, zld, c, expert_of, gate, counters, in ? in->bias : nullptr);
     moe_offsets_kernel<<<1, 32, 0, stream>>>(counters, group_off, E);
     const int n = M * top;
-    moe_scatter_kernel<<<(n + 255) / 256, 256, 0, stream>>>(expert_of, n, top, E, group_off, counters, sorted_tok, slot_of);
+    moe_scatter_kernel<<<(n + 255) / 256, 256, 0, stream>>>(expert_of, n, top, E, group_off, counters, sorted_tok, slot_of,
+                                                            gate, c.slot_gate);
     count_launch(3);
     ASD_CUDA(cudaGetLastError());
     return 0;

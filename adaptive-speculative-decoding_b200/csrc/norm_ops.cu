@@ -184,6 +184,43 @@ __global__ void row_close_kernel(RowClose c) {
     }
 }
 
+// Sublayer close of layers whose norms are tanh(alpha x) w + b: nothing is reduced over a row, so the elements are spread
+// over the grid, V consecutive ones per thread.
+template <int V>
+__global__ void tanh_close_kernel(TanhClose c) {
+    const int m = blockIdx.x, d = (blockIdx.y * blockDim.x + threadIdx.x) * V, D = c.D;
+    if (d >= D) return;
+    const long long base = (long long)m * D + d;
+    float x[V], w[V], b[V];
+    loadv<V>(c.x_in + (c.rows ? (long long)c.rows[m] * D + d : base), x);
+    if (c.y || c.top > 0) {
+        float s[V];
+#pragma unroll
+        for (int e = 0; e < V; ++e) s[e] = 0.f;
+        if (c.y) loadv<V>(c.y + base, s);
+        for (int k = 0; k < c.top; ++k) {       // routed experts' results in choice order
+            float t[V];
+            loadv<V>(c.expert_out + (long long)c.slot_of[(long long)m * c.top + k] * D + d, t);
+#pragma unroll
+            for (int e = 0; e < V; ++e) s[e] += t[e];
+        }
+        const float alpha = *c.post.alpha;
+        loadv<V>(c.post.w + d, w);
+        loadv<V>(c.post.b + d, b);
+#pragma unroll
+        for (int e = 0; e < V; ++e) x[e] = fmaf(c.mult, fmaf(tanhf(alpha * s[e]), w[e], b[e]), x[e]);
+        if (c.x_out) storev<V>(c.x_out + base, x);
+    }
+    if (c.next.w) {
+        const float alpha = *c.next.alpha;
+        loadv<V>(c.next.w + d, w);
+        loadv<V>(c.next.b + d, b);
+#pragma unroll
+        for (int e = 0; e < V; ++e) x[e] = fmaf(tanhf(alpha * x[e]), w[e], b[e]);
+        storevx<V>(c.hn, base, c.hn_f32, x);
+    }
+}
+
 // x[m] = group_norm(embed[token]) * w, fp32 (dynamic shared memory as row_close_kernel)
 __global__ void embed_normed_kernel(SeqIndex ix, const void* embed, int wf32, const float* w, int groups, float eps, float* x,
                                     int D) {
@@ -230,6 +267,31 @@ __global__ void ff_act_kernel(const float* z, void* out, int of32, long long n, 
         if (bias) g += bias[f], u += bias[F + f];
         stx(out, i, of32, g / (1.f + expf(-g)) * u);
     }
+}
+
+// gated activations: z rows of 2 F floats (gate half, then up half), V consecutive results per thread
+template <int V>
+__global__ void gated_act_kernel(const float* z, void* out, int of32, long long rows, int F, GatedAct p) {
+    const int per = F / V;
+    const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= rows * per) return;
+    const long long r = rows * per <= 0x7fffffffLL ? (long long)((unsigned)i / (unsigned)per) : i / per;
+    const int f = (int)(i - r * per) * V;
+    float g[V], u[V];
+    loadv<V>(z + r * 2 * F + f, g);
+    loadv<V>(z + r * 2 * F + F + f, u);
+    const float k = p.row_factor ? p.row_factor[r] : 1.f;
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+        const float ge = g[e] * k, ue = u[e] * k;
+        if (p.kind == GATED_GELU_TANH) {
+            g[e] = gelu_tanh_f(ge) * ue;
+        } else {
+            const float c = fminf(ge, p.limit);
+            g[e] = c / (1.f + expf(-p.slope * c)) * (fminf(fmaxf(ue, -p.limit), p.limit) + 1.f);
+        }
+    }
+    storevx<V>(out, r * F + f, of32, g);
 }
 
 __global__ void rms_rows_kernel(const float* in, long long ld_in, const float* w, int plus_one, float eps, void* out,
@@ -346,6 +408,44 @@ int launch_ff_act(const float* z, void* out, int of32, long long rows, int F, in
     const long long blocks = (n + 255) / 256;
     if (blocks > 0x7fffffffLL) return set_error("ff_act: too many elements");
     ff_act_kernel<<<(unsigned)blocks, 256, 0, stream>>>(z, out, of32, n, F, gated, bias);
+    count_launch(1);
+    ASD_CUDA(cudaGetLastError());
+    return 0;
+}
+
+int launch_gated_act(const float* z, void* out, int of32, long long rows, int F, const GatedAct& p, cudaStream_t stream) {
+    if (rows <= 0 || F <= 0) return 0;
+    if (p.kind == GATED_CLAMPED && !(p.limit > 0.f)) return set_error("gated_act: the limit must be positive");
+    const bool four = F % 4 == 0 && ((reinterpret_cast<uintptr_t>(z) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
+    const long long blocks = (rows * (four ? F / 4 : F) + 255) / 256;
+    if (blocks > 0x7fffffffLL) return set_error("gated_act: too many elements");
+    if (four)
+        gated_act_kernel<4><<<(unsigned)blocks, 256, 0, stream>>>(z, out, of32, rows, F, p);
+    else
+        gated_act_kernel<1><<<(unsigned)blocks, 256, 0, stream>>>(z, out, of32, rows, F, p);
+    count_launch(1);
+    ASD_CUDA(cudaGetLastError());
+    return 0;
+}
+
+int launch_tanh_close(const TanhClose& c, cudaStream_t stream) {
+    if (c.M <= 0) return 0;
+    if (c.D <= 0 || !c.x_in || (c.next.w && !c.hn)) return set_error("tanh_close: bad arguments");
+    if (c.top > 0 && (!c.expert_out || !c.slot_of)) return set_error("tanh_close: expert results missing");
+    if ((c.y || c.top > 0) && (!c.post.w || !c.post.b || !c.post.alpha)) return set_error("tanh_close: the norm of the result is missing");
+    if (c.next.w && (!c.next.b || !c.next.alpha)) return set_error("tanh_close: incomplete norm");
+    uintptr_t at = 0;
+    for (const void* p : {(const void*)c.x_in, (const void*)c.y, (const void*)c.expert_out, (const void*)c.post.w,
+                          (const void*)c.post.b, (const void*)c.x_out, (const void*)c.next.w, (const void*)c.next.b,
+                          (const void*)c.hn})
+        at |= reinterpret_cast<uintptr_t>(p);
+    const bool four = c.D % 4 == 0 && (at & 15) == 0;
+    const int n = four ? c.D / 4 : c.D, threads = n >= 256 ? 256 : (n >= 128 ? 128 : 64);
+    const dim3 grid(c.M, (n + threads - 1) / threads);
+    if (four)
+        tanh_close_kernel<4><<<grid, threads, 0, stream>>>(c);
+    else
+        tanh_close_kernel<1><<<grid, threads, 0, stream>>>(c);
     count_launch(1);
     ASD_CUDA(cudaGetLastError());
     return 0;

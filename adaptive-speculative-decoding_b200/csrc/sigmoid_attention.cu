@@ -178,7 +178,7 @@ __global__ void __launch_bounds__(NT) sigmoid_decode_kernel(MixArgs a) {
 #pragma unroll
         for (int w = 0; w < NW; ++w) t += red[(w * HB + x) * dvp + col];
         if (a.shares == 1) {
-            const float gate = a.gate ? 1.f / (1.f + expf(-a.gate[(long long)m * a.ldg + h])) : 1.f;
+            const float gate = mix_gate(a, m, h, col);
             stx(a.out, (long long)m * a.ldo + (long long)h * dv + col, a.of32, t * gate);
         } else {
             a.part[((long long)share * M + m) * H * dv + (long long)h * dv + col] = t;

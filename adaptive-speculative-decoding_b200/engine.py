@@ -10,7 +10,8 @@ from typing import Dict, Optional
 
 import torch
 
-from ._lib import (AsdError, DikopelConfigC, DikopelLayerC, LukopelConfigC, LukopelLayerC, MavipelConfigC, MavipelLayerC, MezilixConfigC, MezilixLayerC, ModelConfigC, RivetarConfigC,
+from ._lib import (AsdError, DikopelConfigC, DikopelLayerC, LukopelConfigC, LukopelLayerC, MavipelConfigC, MavipelLayerC, MezilixConfigC, MezilixLayerC, ModelConfigC,
+                   NobonexConfigC, NobonexLayerC, RivetarConfigC,
                    RivetarLayerC, check, lib)
 from .models.qwen2 import Qwen2Config, pack_layer, random_packed_layer
 from .ops import NUM_FEATURES
@@ -821,6 +822,36 @@ class DikopelEngine(RivetarEngine):
                                    l.a_dim, l.a_vdim, l.r_heads, l.r_kv_heads, l.r_dim, l.r_vdim, l.conv,
                                    self.FF_CODE[l.ff_kind], l.ff, l.experts, l.top, l.expert_ff, l.shared_ff, l.groups,
                                    l.keep, l.gate_cap, l.scale, l.router_scale)
+        return c, arr
+
+
+class NobonexEngine(RivetarEngine):
+    """One Nobonex-family model on one GPU: wraps an ``asd_nobonex_engine_t`` handle.  Same ownership as
+    ``RivetarEngine``: the paged key/value caches of the attention layers (``PageTable``; a layer that reads another
+    layer's keys and values has none of its own) and, in one fp32 buffer, the carried inputs of the convolutions and the
+    recurrent states, one entry per ring position; entry position % ring is the state after that position, and a forward
+    that starts a slot at position 0 starts from zero, so reused slots carry nothing over.  Same ``forward`` interface as
+    ``QwenEngine``, so ``SpecDecoder``, ``Stage`` and the trace runner drive it unchanged."""
+
+    TYPE_CODE = {"attention": 0, "mamba2": 1, "attention_2": 2}
+    FF_CODE = {None: 0, "dense": 1, "moe": 2}
+    PREFIX = "nobonex"
+    PROFILE_CLASSES = ("dense", "attention", "recurrence", "experts", "router", "activation", "glue", "lm_head")
+
+    @staticmethod
+    def _family():
+        from .models import nobonex
+        return nobonex
+
+    def _c_config(self, cfg, max_tokens: int, page_size: int, dtype):
+        c = NobonexConfigC(cfg.width, cfg.vocab_size, cfg.num_hidden_layers, cfg.eps, cfg.embed_scale, cfg.residual_mult,
+                           max_tokens, page_size, self.ring, 1 if dtype == torch.float32 else 0)
+        arr = (NobonexLayerC * max(1, cfg.num_hidden_layers))()
+        for i, l in enumerate(cfg.layers):
+            y = l.yarn or (0.0, 0.0, 0.0, 0.0)
+            arr[i] = NobonexLayerC(self.TYPE_CODE[l.type], l.kv_from, l.heads, l.kv_heads, l.dim, l.vdim, l.conv, l.rot_dims,
+                                   min(l.chunk, 1 << 30), l.state, l.groups, l.norm_groups, self.FF_CODE[l.ff_kind], l.ff,
+                                   l.experts, l.top, l.expert_ff, l.scale, l.softcap, l.limit, l.rot_base, *y)
         return c, arr
 
 

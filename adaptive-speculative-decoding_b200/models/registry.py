@@ -1,7 +1,7 @@
 """Model registry: which configuration class, engine class and library components serve a checkpoint.
 
 A checkpoint directory is recognised by its ``config.json``: ``"architecture": "Mezilix"`` / ``"Rivetar"`` /
-``"Mavipel"`` / ``"Lukopel"`` / ``"Dikopel"`` or the Hugging Face keys ``architectures`` / ``model_type`` of the Qwen2
+``"Mavipel"`` / ``"Lukopel"`` / ``"Dikopel"`` / ``"Nobonex"`` or the Hugging Face keys ``architectures`` / ``model_type`` of the Qwen2
 family (what the reference hands to vLLM, src/serving/real_model_pipeline.py:98-108).  ``Stage``, the trace runner and ``bench.py`` all go through here."""
 from __future__ import annotations
 
@@ -55,6 +55,11 @@ def _dikopel_cfg(d: dict, name: str = "dikopel"):
     return DikopelConfig.from_dict(d, name=name)
 
 
+def _nobonex_cfg(d: dict, name: str = "nobonex"):
+    from .nobonex import NobonexConfig
+    return NobonexConfig.from_dict(d, name=name)
+
+
 def _qwen_engine():
     from ..engine import QwenEngine
     return QwenEngine
@@ -85,6 +90,11 @@ def _dikopel_engine():
     return DikopelEngine
 
 
+def _nobonex_engine():
+    from ..engine import NobonexEngine
+    return NobonexEngine
+
+
 FAMILIES: Dict[str, Family] = {
     "qwen2": Family("qwen2", ("linear", "qwen", "sampling"), ("bfloat16",), _qwen_cfg, _qwen_engine),
     "mezilix": Family("mezilix", ("mezilix",), ("bfloat16", "float32"), _mezilix_cfg, _mezilix_engine),
@@ -92,6 +102,7 @@ FAMILIES: Dict[str, Family] = {
     "mavipel": Family("mavipel", ("mavipel",), ("bfloat16", "float32"), _mavipel_cfg, _mavipel_engine),
     "lukopel": Family("lukopel", ("lukopel",), ("bfloat16", "float32"), _lukopel_cfg, _lukopel_engine),
     "dikopel": Family("dikopel", ("dikopel",), ("bfloat16", "float32"), _dikopel_cfg, _dikopel_engine),
+    "nobonex": Family("nobonex", ("nobonex",), ("bfloat16", "float32"), _nobonex_cfg, _nobonex_engine),
 }
 
 

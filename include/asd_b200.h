@@ -621,6 +621,83 @@ ASD_API int asd_dikopel_forward(asd_dikopel_engine_t* e, const int32_t* tokens, 
 ASD_API int asd_dikopel_profile_read(asd_dikopel_engine_t* e, float* ms_by_class, int* launches_by_class, int nclass);
 ASD_API int asd_dikopel_device_error(asd_dikopel_engine_t* e);
 
+/* ------------------------------------------------------------------------------------------------------------------
+ * Nobonex family engine (nobonex_engine.cu).  x = embed[token] * embed_scale.  Every layer norms before and after each
+ * sublayer: x <- x + residual_mult * norm1b(mixer(norm1(x))); x <- x + residual_mult * norm2b(ff(norm2(x))).
+ * logits = head . final_norm(x).  A norm is a dynamic tanh, N(x) = tanh(alpha x) * w + b with one alpha per norm.  Mixers:
+ *   type 0  convolved attention (heads, kv_heads, dim = vdim): q and k pass a causal convolution over time (conv taps per
+ *           channel, no bias, no activation); a convolved key is the value; q and k are then RMS-normed over the whole
+ *           projection (eps) and rotated over the leading rot_dims coordinates of each head in pairs (2i, 2i + 1);
+ *           causal softmax attention over scale * q . k;
+ *   type 1  scalar-decay state space recurrence: projection [z | x | B | C | dt] with z, x heads * vdim, B, C groups * state,
+ *           dt heads values; x, B, C pass a causal convolution with bias and silu; dt <- softplus(dt + dt_bias);
+ *           S <- exp(-exp(a_log) dt) S + dt B x^T, y = S^T C + skip x per head; y * silu(z) is RMS-normed in norm_groups equal
+ *           parts, times out_norm;
+ *   type 2  chunked attention (heads, kv_heads, dim, vdim): biased projections, RMS norm per head, rotation in pairs
+ *           (i, i + rot_dims/2), scores scale * q . k capped as softcap * tanh(. / softcap) (0: not), position i sees j <= i
+ *           with i / chunk == j / chunk (chunk 0: every j <= i), softmax; the result times sigmoid of a projection of the
+ *           mixer's input, element by element.  kv_from >= 0: keys and values are those of that earlier layer of type 2.
+ * Rotation: angle = position * rot_base^(-2i/rot_dims); yarn_factor > 0 rescales the frequencies (pairs between those that
+ * turn yarn_fast and yarn_slow times over yarn_original positions by a linear ramp to 1 / factor) and multiplies cos and sin by
+ * 0.1 ln(factor) + 1.
+ * ff_kind 0: none; 1: W_down (gelu_tanh(W_gate h) * W_up h); 2: `experts` layers of size expert_ff of which every token takes
+ * the `top` with the largest sigmoid(router logit), each on its input times that score: g = min(W_gate h, limit),
+ * u = clamp(W_up h, +-limit), W_down (g sigmoid(1.702 g) (u + 1)), summed.
+ *
+ * dtype as for the Rivetar engine.  Paged pool: per layer of type 0 or 2 without kv_from [num_pages][page_size][kv_heads *
+ * (dim + vdim)], keys then values, layers back to back.  State (caller allocated, fp32), per layer: carried inputs of the
+ * convolution [max_seqs][conv - 1 + ring - 1][channels] (types 0 and 1), then [max_seqs][ring][heads][state][vdim] (type 1),
+ * every one of these parts starting on a 16-byte boundary; entry position % ring holds the state AFTER that position, so a
+ * caller may re-feed any of the last `ring` positions; a run that starts at position 0 starts from zero.
+ */
+typedef struct asd_nobonex_layer_config {
+    int type;                                       /* 0 convolved attention, 1 state space, 2 chunked attention */
+    int kv_from;                                    /* type 2: -1 or the layer whose keys and values are used */
+    int heads, kv_heads, dim, vdim;                 /* type 1: heads and vdim */
+    int conv, rot_dims, chunk;
+    int state, groups, norm_groups;                 /* type 1 */
+    int ff_kind, ff, experts, top, expert_ff;
+    float scale, softcap, limit;
+    double rot_base, yarn_factor, yarn_original, yarn_fast, yarn_slow;
+} asd_nobonex_layer_config;
+typedef struct asd_nobonex_config {
+    int width, vocab, n_layers;
+    float eps, embed_scale, residual_mult;
+    int max_tokens, page_size, ring, dtype;
+} asd_nobonex_config;
+typedef struct asd_nobonex_engine asd_nobonex_engine_t;
+
+ASD_API asd_nobonex_engine_t* asd_nobonex_create(const asd_nobonex_config* cfg, const asd_nobonex_layer_config* layers);
+ASD_API void asd_nobonex_destroy(asd_nobonex_engine_t* e);
+/* Weights by name; matrices row-major [out, in] in the engine's dtype, vectors and everything marked fp32 always fp32.
+ * layer -1: "embed" [vocab, width], "final_norm", "final_norm_b" [width], "final_norm_alpha" [1], "head" [vocab, width].
+ * Every layer: "norm1", "norm1_b", "norm1_alpha", "norm1b", "norm1b_b", "norm1b_alpha", and with a feed-forward the same with
+ * norm2; "w_in" = the matrices that read the mixer input stacked by rows, "w_o" = the output projection:
+ *   type 0: w_in [q | k]; "q_norm" [heads * dim], "k_norm" [kv_heads * dim], "conv_w" fp32 [q, k channels][conv];
+ *   type 1: w_in [z | x | B | C | dt]; "conv_w" fp32 [x, B, C channels][conv], "conv_b", "a_log", "dt_bias", "skip" [heads],
+ *           "out_norm" [heads * vdim];
+ *   type 2: w_in [q | k | v | gate] (kv_from: [q | gate]); "in_bias" [q, k, v rows] (kv_from: [q rows]), "q_norm", "k_norm"
+ *           [dim] (kv_from: q_norm alone).
+ * ff_kind 1: "w_gu" [2 ff, width] (gate rows, then up rows), "w_down" [width, ff].  ff_kind 2: "router" fp32 [experts, width],
+ * "w_egu" [experts][2 expert_ff, width], "w_edown" [experts][width, expert_ff]. */
+ASD_API int asd_nobonex_set_tensor(asd_nobonex_engine_t* e, int layer, const char* name, const void* data);
+ASD_API size_t asd_nobonex_cache_bytes(const asd_nobonex_engine_t* e, int num_pages);
+ASD_API size_t asd_nobonex_state_bytes(const asd_nobonex_engine_t* e, int max_seqs);
+ASD_API int asd_nobonex_set_cache(asd_nobonex_engine_t* e, void* pool, int num_pages, const int32_t* page_table,
+                                  int max_seqs, int max_pages_per_seq, float* state);
+/* options: "tc_linear", "tc_min_rows", "attn_general", "profile" as for the Dikopel engine; "ssd_mode" 0: prompts of a bf16
+ * engine run the recurrence chunk by chunk on the tensor cores, 1: position by position in fp32 */
+ASD_API int asd_nobonex_set_option(asd_nobonex_engine_t* e, const char* name, int value);
+/* Same arguments as asd_engine_forward (M <= max_tokens).  layer_out (optional, fp32 [n_layers][M][width]) receives the
+ * stream that leaves every layer. */
+ASD_API int asd_nobonex_forward(asd_nobonex_engine_t* e, const int32_t* tokens, const int32_t* positions,
+                                const int32_t* token_slot, int M, const int32_t* cu_q, const int32_t* seq_slot, int nseq,
+                                int max_qlen, int max_kv_len, const int32_t* logit_rows, int n_logit_rows,
+                                float* logits_out, long long logits_ld, float* layer_out, void* stream);
+/* ms and launches by kernel class since the last read (nclass >= 8), classes as for the Dikopel engine */
+ASD_API int asd_nobonex_profile_read(asd_nobonex_engine_t* e, float* ms_by_class, int* launches_by_class, int nclass);
+ASD_API int asd_nobonex_device_error(asd_nobonex_engine_t* e);
+
 #ifdef __cplusplus
 }
 #endif
