@@ -34,7 +34,7 @@ COMPONENTS = {
     "mavipel": ["mavipel_engine.cu", "talking_attention.cu"],
     "lukopel": ["lukopel_engine.cu", "residual_streams.cu"],
     "dikopel": ["dikopel_engine.cu", "mlstm.cu"],
-    "nobonex": ["nobonex_engine.cu", "ssd.cu"],
+    "nobonex": ["nobonex_engine.cu", "ssd.cu", "ssd_chunk.cu"],
     "qwen": ["engine.cu", "layers.cu", "attention.cu", "attention_tc.cu", "forward_persist.cu"],
     "sampling": ["api.cu", "sampler.cu", "stop_rule.cu"],
 }

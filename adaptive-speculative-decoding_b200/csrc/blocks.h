@@ -506,10 +506,11 @@ struct SsdDims {
     int heads, groups, dk, dv;
 };
 struct SsdInput {
-    const float* x = nullptr;    // fp32 rows ld floats apart: heads * dv used
-    const float* b = nullptr;    // groups * dk used
-    const float* c = nullptr;
+    const void* x = nullptr;     // rows ld elements apart: heads * dv used
+    const void* b = nullptr;     // groups * dk used
+    const void* c = nullptr;
     long long ld = 0;
+    int bf16 = 0;                // element type of x, b and c: 1 bf16, 0 fp32
     const float* dt = nullptr;   // raw, fp32 rows ld_dt apart: one per head
     long long ld_dt = 0;
     const float* dt_bias = nullptr;   // [heads] each
@@ -518,8 +519,8 @@ struct SsdInput {
 };
 // state fp32 [slots][ring][heads][dk][dv]; entry position % ring holds the state after that position.  A sequence whose
 // first new position is 0 starts from zero, any other from entry (position - 1) % ring; the last `ring` new positions of
-// a sequence store theirs.  out fp32 [M][heads * dv].  mode 0: prompts run chunk by chunk on the tensor cores (fp32 operands
-// as two bf16 terms, fp32 state) where the sizes allow; 1: position by position in fp32.
+// a sequence store theirs.  out fp32 [M][heads * dv].  mode 0: prompts with bf16 inputs run chunk by chunk on the tensor
+// cores (fp32 operands as two bf16 terms, fp32 state) where the sizes allow; 1: position by position in fp32.
 int launch_ssd_recurrence(const SeqIndex& ix, const int* cu_q, const int* seq_slot, int nseq, int max_qlen, const SsdInput& in,
                           const SsdDims& d, float* state, int ring, float* out, int mode, cudaStream_t stream);
 

@@ -585,9 +585,11 @@ __global__ void head_norm_gate_kernel(const float* o, HeadNormGate p, void* y, i
     for (int i = lane; i < dv; i += 32) stx(y, m * ldy + (long long)h * dv + i, of32, src[i] * r * w[i] * gate(i));
 }
 
-// parts too long for a warp: a CTA each, its gated values kept in registers between the sum and the result
-constexpr int WIDE_T = 256, WIDE_V = 8;
-__global__ void __launch_bounds__(WIDE_T) part_norm_gate_kernel(const float* o, HeadNormGate p, void* y, int of32, long long ldy,
+// parts too long for a warp: a CTA each, four consecutive elements a thread, U blocks of them kept in registers between the
+// sum of squares and the result
+constexpr int PART_T = 256;
+template <int U>
+__global__ void __launch_bounds__(PART_T) part_norm_gate_kernel(const float* o, HeadNormGate p, void* y, int of32, long long ldy,
                                                                 int heads, int dv) {
     __shared__ float red[33];
     const int h = blockIdx.y;
@@ -595,23 +597,33 @@ __global__ void __launch_bounds__(WIDE_T) part_norm_gate_kernel(const float* o, 
     const float* src = o + (m * heads + h) * dv;
     const float* g = p.gate + m * p.ldg + (long long)h * dv;
     const float* w = p.w + (p.w_per_head ? (long long)h * dv : 0);
-    float v[WIDE_V], gv[WIDE_V];
+    float v[U][4];
     float ss = 0.f;
 #pragma unroll
-    for (int u = 0; u < WIDE_V; ++u) {
-        const int i = u * WIDE_T + threadIdx.x;
-        v[u] = gv[u] = 0.f;
-        if (i >= dv) continue;
-        v[u] = src[i], gv[u] = g[i];
-        if (p.gate_act) gv[u] = (p.gate_act == 2 ? gv[u] : 1.f) * sigmoid_f(gv[u]);
-        const float t = p.gate_first ? v[u] * gv[u] : v[u];
-        ss = fmaf(t, t, ss);
+    for (int u = 0; u < U; ++u) {
+        const int i = (u * PART_T + threadIdx.x) * 4;
+        float gv[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+        for (int e = 0; e < 4; ++e) v[u][e] = 0.f;
+        if (i < dv) ldx4(src, i, 1, v[u]), ldx4(g, i, 1, gv);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const float gt = p.gate_act ? (p.gate_act == 2 ? gv[e] : 1.f) * sigmoid_f(gv[e]) : gv[e];
+            const float t = v[u][e] * gt;
+            ss = p.gate_first ? fmaf(t, t, ss) : fmaf(v[u][e], v[u][e], ss);
+            v[u][e] = t;
+        }
     }
     const float r = p.scale / sqrtf(block_sum(ss, red) / (float)dv + p.eps);
 #pragma unroll
-    for (int u = 0; u < WIDE_V; ++u) {
-        const int i = u * WIDE_T + threadIdx.x;
-        if (i < dv) stx(y, m * ldy + (long long)h * dv + i, of32, v[u] * r * w[i] * gv[u]);
+    for (int u = 0; u < U; ++u) {
+        const int i = (u * PART_T + threadIdx.x) * 4;
+        if (i >= dv) continue;
+        float wv[4];
+        ldx4(w, i, 1, wv);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) v[u][e] *= r * wv[e];
+        stx4(y, m * ldy + (long long)h * dv + i, of32, v[u]);
     }
 }
 
@@ -790,8 +802,14 @@ int launch_head_norm_gate(const float* o, const HeadNormGate& p, void* y, int of
                           cudaStream_t stream) {
     if (M <= 0) return 0;
     if (!p.w || !p.gate) return set_error("head_norm_gate: missing inputs");
-    if (dv > 512 && dv <= WIDE_T * WIDE_V && heads <= 65535) {
-        part_norm_gate_kernel<<<dim3(M, heads), WIDE_T, 0, stream>>>(o, p, y, of32, ldy, heads, dv);
+    uintptr_t at = 0;
+    for (const void* q : {(const void*)o, (const void*)p.gate, (const void*)p.w, (const void*)y}) at |= reinterpret_cast<uintptr_t>(q);
+    if (dv > 512 && dv % 4 == 0 && dv <= 16 * 4 * PART_T && p.ldg % 4 == 0 && ldy % 4 == 0 && (at & 15) == 0 && heads <= 65535) {
+        const dim3 grid(M, heads);
+        const int u = (dv + 4 * PART_T - 1) / (4 * PART_T);
+        auto run = [&](auto kernel) { kernel<<<grid, PART_T, 0, stream>>>(o, p, y, of32, ldy, heads, dv); };
+        u <= 1 ? run(part_norm_gate_kernel<1>) : u <= 2 ? run(part_norm_gate_kernel<2>) : u <= 4 ? run(part_norm_gate_kernel<4>)
+               : u <= 8 ? run(part_norm_gate_kernel<8>) : run(part_norm_gate_kernel<16>);
         count_launch(1);
         ASD_CUDA(cudaGetLastError());
         return 0;

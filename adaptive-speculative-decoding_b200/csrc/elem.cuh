@@ -41,6 +41,16 @@ __device__ __forceinline__ void stx(void* p, long long i, int f32, float v) {
     else
         ((__nv_bfloat16*)p)[i] = __float2bfloat16(v);
 }
+// four consecutive elements to a place that is a multiple of four in a 16-byte aligned buffer
+__device__ __forceinline__ void stx4(void* p, long long i, int f32, const float (&v)[4]) {
+    if (f32) {
+        *reinterpret_cast<float4*>((float*)p + i) = make_float4(v[0], v[1], v[2], v[3]);
+    } else {
+        __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
+        *reinterpret_cast<uint2*>((__nv_bfloat16*)p + i) =
+            make_uint2(*reinterpret_cast<uint32_t*>(&lo), *reinterpret_cast<uint32_t*>(&hi));
+    }
+}
 
 // two fp32 operations in one instruction (each rounded as its scalar form)
 __device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {

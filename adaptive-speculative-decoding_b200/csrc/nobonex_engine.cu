@@ -171,17 +171,19 @@ static int mix_ssd(NbEngine* e, const NbLayer& ly, int li, const Batch& b, cudaS
     {
         NB_PROF(NB_GLUE);
         if (launch_carried_conv(b.ix, b.cu_q, b.nseq, b.max_qlen, e->proj + inner, ly.ld_in, ly.f("conv_w"), c.conv, ly.conv_ch,
-                                e->state + ly.conv_off, ly.conv_ring, CONV_SILU, e->conv, 1, s, ly.f("conv_b")))
+                                e->state + ly.conv_off, ly.conv_ring, CONV_SILU, e->conv, e->f32, s, ly.f("conv_b")))
             return -1;
     }
     {
         NB_PROF(NB_RECUR);
         SsdInput in;
-        in.x = e->conv, in.b = e->conv + inner, in.c = in.b + bc, in.ld = ly.conv_ch;
+        char* cv = reinterpret_cast<char*>(e->conv);
+        in.x = cv, in.b = cv + (size_t)inner * e->esz, in.c = cv + (size_t)(inner + bc) * e->esz, in.ld = ly.conv_ch;
+        in.bf16 = !e->f32;
         in.dt = e->proj + inner + ly.conv_ch, in.ld_dt = ly.ld_in;
         in.dt_bias = ly.f("dt_bias"), in.a_log = ly.f("a_log"), in.skip = ly.f("skip");
         if (launch_ssd_recurrence(b.ix, b.cu_q, b.seq_slot, b.nseq, b.max_qlen, in, SsdDims{c.heads, c.groups, c.state, c.vdim},
-                                  e->state + ly.state_off, e->c.ring, e->orec, e->f32 ? 1 : e->ssd_mode, s))
+                                  e->state + ly.state_off, e->c.ring, e->orec, e->ssd_mode, s))
             return -1;
     }
     {

@@ -9,6 +9,8 @@
 #include <cuda_bf16.h>
 #include <math.h>
 
+#include <algorithm>
+
 #include "asd_internal.h"
 #include "blocks.h"
 #include "elem.cuh"
@@ -41,7 +43,7 @@ template <int ROWS, int MAXT>
 __global__ void __launch_bounds__(MAXT, 1) ssd_recurrence_kernel(SsdArgs a) {
     extern __shared__ __align__(16) float sm[];
     const int seq = blockIdx.x, head = blockIdx.y, col0 = blockIdx.z * 32;
-    const int t0 = a.cu_q[seq], t1 = a.cu_q[seq + 1];
+    const int t1 = a.cu_q[seq + 1], t0 = a.tail > 0 ? max(a.cu_q[seq], t1 - a.tail) : a.cu_q[seq];
     if (t0 >= t1) return;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, RS = blockDim.x >> 5, nthr = blockDim.x;
     const int dk = a.d.dk, dv = a.d.dv, H = a.d.heads, CH = a.CH, ring = a.ring;
@@ -76,26 +78,37 @@ __global__ void __launch_bounds__(MAXT, 1) ssd_recurrence_kernel(SsdArgs a) {
         float* bs = cs + CH * dkp;
         float* xs = bs + CH * dkp;
         float* ds = xs + CH * 32;
-        if (a.v16) {
+        if (a.in.bf16) {
+            for (int i = threadIdx.x; i < nt * dk; i += nthr) {
+                const int t = i / dk, c = i - t * dk;
+                const long long at = (long long)(c0 + t) * a.in.ld + (long long)grp * dk + c;
+                cs[t * dkp + c] = ssd_in(a, a.in.c, at);
+                bs[t * dkp + c] = ssd_in(a, a.in.b, at);
+            }
+        } else if (a.v16) {
             const int n4 = dk >> 2;
             for (int i = threadIdx.x; i < nt * n4; i += nthr) {
                 const int t = i / n4, c = (i - t * n4) * 4;
                 const long long at = (long long)(c0 + t) * a.in.ld + (long long)grp * dk + c;
-                stage16(cs + t * dkp + c, a.in.c + at);
-                stage16(bs + t * dkp + c, a.in.b + at);
+                stage16(cs + t * dkp + c, static_cast<const float*>(a.in.c) + at);
+                stage16(bs + t * dkp + c, static_cast<const float*>(a.in.b) + at);
             }
         } else {
             for (int i = threadIdx.x; i < nt * dk; i += nthr) {
                 const int t = i / dk, c = i - t * dk;
                 const long long at = (long long)(c0 + t) * a.in.ld + (long long)grp * dk + c;
-                stage4(cs + t * dkp + c, a.in.c + at, true);
-                stage4(bs + t * dkp + c, a.in.b + at, true);
+                stage4(cs + t * dkp + c, static_cast<const float*>(a.in.c) + at, true);
+                stage4(bs + t * dkp + c, static_cast<const float*>(a.in.b) + at, true);
             }
         }
         for (int i = threadIdx.x; i < nt * 32; i += nthr) {
             const int t = i >> 5, c = i & 31;
             const bool ok = col0 + c < dv;
-            stage4(xs + i, a.in.x + (ok ? (long long)(c0 + t) * a.in.ld + (long long)head * dv + col0 + c : 0), ok);
+            const long long at = ok ? (long long)(c0 + t) * a.in.ld + (long long)head * dv + col0 + c : 0;
+            if (a.in.bf16)
+                xs[i] = ok ? ssd_in(a, a.in.x, at) : 0.f;
+            else
+                stage4(xs + i, static_cast<const float*>(a.in.x) + at, ok);
         }
         for (int t = threadIdx.x; t < nt; t += nthr) stage4(ds + t, a.in.dt + (long long)(c0 + t) * a.in.ld_dt + head, true);
         asm volatile("cp.async.commit_group;" ::: "memory");
@@ -195,16 +208,16 @@ __global__ void __launch_bounds__(ST) ssd_step_kernel(SsdArgs a) {
     load(rg);
     const long long row = (long long)m * a.in.ld;
     for (int i = tid; i < dk; i += ST) {
-        cs[i] = a.in.c[row + (long long)grp * dk + i];
-        bs[i] = a.in.b[row + (long long)grp * dk + i];
+        cs[i] = ssd_in(a, a.in.c, row + (long long)grp * dk + i);
+        bs[i] = ssd_in(a, a.in.b, row + (long long)grp * dk + i);
     }
     const float dt = softplus_step(a.in.dt[(long long)m * a.in.ld_dt + head] + a.in.dt_bias[head]);
     const float keep = 1.f + expm1f(-expf(a.in.a_log[head]) * dt);
-    const float* x = a.in.x + row + (long long)head * dv + col0;
+    const long long x_at = row + (long long)head * dv + col0;
     float xv[4] = {0.f, 0.f, 0.f, 0.f}, o[4] = {0.f, 0.f, 0.f, 0.f};
     if (live)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) xv[e] = dt * x[c4 + e];
+        for (int e = 0; e < 4; ++e) xv[e] = dt * ssd_in(a, a.in.x, x_at + c4 + e);
     __syncthreads();
     for (int r0 = rg; r0 < dk && live; r0 += SU * R) {
         if (r0 != rg) load(r0);
@@ -229,7 +242,7 @@ __global__ void __launch_bounds__(ST) ssd_step_kernel(SsdArgs a) {
     for (int c = tid; c < 4 * L; c += ST) {
         float t = 0.f;
         for (int r = 0; r < R; ++r) t += red[r * 4 * L + c];
-        a.out[(long long)m * H * dv + (long long)head * dv + col0 + c] = fmaf(skip, x[c], t);
+        a.out[(long long)m * H * dv + (long long)head * dv + col0 + c] = fmaf(skip, ssd_in(a, a.in.x, x_at + c), t);
     }
 }
 
@@ -253,12 +266,21 @@ int launch_ssd_recurrence(const SeqIndex& ix, const int* cu_q, const int* seq_sl
         ASD_CUDA(cudaGetLastError());
         return 0;
     }
-    (void)mode;
+    if (mode == 0 && in.bf16 && max_qlen >= 16) {
+        // chunks leave the state after their last position; the states of the ring's other entries come from a sequential
+        // pass over the last positions
+        a.tail = ring - 1;
+        const int rc = launch_ssd_chunks(a, nseq, stream);
+        if (rc < 0) return -1;
+        if (rc == 0 && ring == 1) return 0;
+        if (rc == 1) a.tail = 0;
+    }
     int rows = 4;
     while (rows < 32 && rows * 4 < d.dk) rows *= 2;     // four warps up to key size 128, then more
     const int RS = (d.dk + rows - 1) / rows, dkp = RS * rows;
     int ch = MAXC;   // positions per staged chunk; steps of few tokens stage (and clear) no more than they use
-    while (ch > 1 && (long long)(ch / 2) * nseq >= ix.M) ch >>= 1;
+    const long long positions = a.tail > 0 ? std::min<long long>(ix.M, (long long)nseq * a.tail) : ix.M;
+    while (ch > 1 && (long long)(ch / 2) * nseq >= positions) ch >>= 1;
     auto need = [&](int c) { return (size_t)total_floats(c, dkp, RS) * sizeof(float); };
     while (ch > 1 && need(ch) > 112 * 1024) ch >>= 1;
     const size_t smem = need(ch);

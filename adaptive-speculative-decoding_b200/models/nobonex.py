@@ -15,7 +15,7 @@ from __future__ import annotations
 import json
 import math
 import os
-from dataclasses import dataclass, field
+from dataclasses import dataclass, field, replace
 from typing import Dict, List, Optional, Tuple
 
 import torch
@@ -264,10 +264,10 @@ def tiny_config(**kw) -> NobonexConfig:
 
 def sized_config(width: int, n_layers: int, heads: int, vocab: int = 32768, dim: int = 128, chunk: int = 1024,
                  ff: Optional[int] = None, experts: int = 0, top: int = 2, name: str = "nobonex-sized") -> NobonexConfig:
-    """layers of a realistic size for throughput measurements (random weights): two state space layers (2 x width inner values
-    in heads of 64, state 128), an attention layer, two more, then a chunked attention layer, in turn; every second chunked
-    layer reads the first one's keys and values.  Dense feed-forwards of width ff (3 x width by default), or `experts`
-    experts of ff / (top + 1)"""
+    """layers of a realistic size for throughput measurements (random weights), six in turn: state space (2 x width inner
+    values in heads of 64, state 128) twice, convolved attention, state space, chunked attention, chunked attention with the
+    keys and values of the one before.  Dense feed-forwards of width ff (3 x width by default), or `experts` experts of
+    ff / (top + 1)"""
     ff = ff if ff is not None else 3 * width
     f = dict(ff_kind="moe", experts=experts, top=top, expert_ff=max(64, ff // (top + 1)), limit=7.0) if experts else \
         dict(ff_kind="dense", ff=ff)
@@ -275,17 +275,10 @@ def sized_config(width: int, n_layers: int, heads: int, vocab: int = 32768, dim:
     rot = dict(rot_dims=dim // 2, rot_base=500000.0)
     ssd = NobonexLayer(type="mamba2", heads=2 * width // 64, vdim=64, state=128, groups=1, norm_groups=1, conv=4, **f)
     att = NobonexLayer(type="attention", heads=heads, kv_heads=kv, dim=dim, vdim=dim, scale=dim ** -0.5, conv=4, **rot, **f)
-    layers: List[NobonexLayer] = []
-    source = -1
-    for i in range(n_layers):
-        if i % 3 != 2:
-            layers.append(ssd)
-        elif i % 6 == 2:
-            layers.append(att)
-        else:
-            layers.append(NobonexLayer(type="attention_2", heads=heads, kv_heads=kv, dim=dim, vdim=dim, scale=dim ** -0.5,
-                                       yarn=(4.0, 4096.0, 32.0, 1.0), chunk=chunk, softcap=50.0, kv_from=source, **rot, **f))
-            source = i if source < 0 else source
+    chk = NobonexLayer(type="attention_2", heads=heads, kv_heads=kv, dim=dim, vdim=dim, scale=dim ** -0.5,
+                       yarn=(4.0, 4096.0, 32.0, 1.0), chunk=chunk, softcap=50.0, **rot, **f)
+    cycle = (ssd, ssd, att, ssd, chk, chk)
+    layers = [replace(cycle[i % 6], kv_from=i - 1) if i % 6 == 5 else cycle[i % 6] for i in range(n_layers)]
     return NobonexConfig(width=width, vocab_size=vocab, layers=layers, embed_scale=1.0, residual_mult=0.5, name=name)
 
 

@@ -674,7 +674,7 @@ def family_sizes(family="mezilix"):
     """(label, configuration of the family, configuration it is measured beside: for Mezilix and Rivetar a Qwen2 model of
     the same width, depth, head count and active weights per layer; for Mavipel the Rivetar model of the same width,
     depth and head count, whose recurrence and windowed attention are the like kernels; for Lukopel and Dikopel the Mavipel
-    model of the same width, depth and head count)"""
+    model and for Nobonex the Dikopel model of the same width, depth and head count)"""
     from asd_b200.models.qwen2 import Qwen2Config
     out = []
     for label, width, heads, layers in (("w2048", 2048, 16, 4), ("w4096", 4096, 32, 4)):
@@ -695,6 +695,15 @@ def family_sizes(family="mezilix"):
             mv = mavipel.sized_config(width, layers, heads, vocab=32768, dim=128, window=1024, ff=3 * width,
                                       name=f"mavipel-{label}")
             out.append((label, fm, mv))
+            continue
+        if family == "nobonex":
+            from asd_b200.models import dikopel, nobonex
+            layers = 6          # three state space layers, convolved attention, chunked attention, chunked with shared keys
+            fm = nobonex.sized_config(width, layers, heads, vocab=32768, dim=128, chunk=1024, ff=3 * width, experts=8, top=2,
+                                      name=f"nobonex-{label}")
+            dk = dikopel.sized_config(width, layers, heads, vocab=32768, dim=128, ff=3 * width, experts=8, top=2,
+                                      name=f"dikopel-{label}")
+            out.append((label, fm, dk))
             continue
         if family == "dikopel":
             from asd_b200.models import dikopel, mavipel
@@ -871,14 +880,47 @@ def dikopel_model(cfg, M, kv_len, nseq):
     return {k: tuple(v) for k, v in cls.items()}
 
 
+def nobonex_model(cfg, M, kv_len, nseq):
+    """algorithmic (FLOPs, bytes) of one forward per kernel class, summed over the layers (bf16 engine).  Recurrence: 5
+    operations per state element and position as the rule is written; bytes = the state in and out once per sequence plus a
+    position's vectors.  Attention: the visible cache rows once per sequence and layer (also a layer that reads another's)."""
+    D = cfg.width
+    tri = 0.5 if M > nseq else 1.0
+    cls = {k: [0.0, 0.0] for k in ("dense", "attention", "recurrence", "experts")}
+
+    def add(k, fl, by):
+        cls[k][0] += fl
+        cls[k][1] += by
+    for l in cfg.layers:
+        nv = l.heads * l.vdim
+        if l.type == "mamba2":
+            add("recurrence", 5.0 * M * l.state_elems, 8.0 * nseq * l.state_elems + 4.0 * M * (l.conv_channels + nv))
+        else:
+            keys = min(l.chunk, kv_len) if l.chunk else kv_len
+            kvw = l.kv_heads * (l.dim + l.vdim)
+            add("attention", 2.0 * M * l.heads * keys * (l.dim + l.vdim) * tri,
+                2.0 * nseq * (kv_len if M > nseq else keys) * kvw + 4.0 * M * l.heads * l.dim + 2.0 * M * nv)
+        wd = (l.in_rows + nv) * D
+        act = M * (2 * D + 4 * l.in_rows + 2 * nv + 4 * D)
+        if l.ff_kind == "dense":
+            wd += 3 * l.ff * D
+            act += M * (2 * D + 10 * l.ff + 4 * D)
+        elif l.ff_kind == "moe":
+            hit = l.experts * (1.0 - (1.0 - l.top / l.experts) ** M)
+            add("experts", 2.0 * M * l.top * 3 * l.expert_ff * D,
+                2.0 * hit * 3 * l.expert_ff * D + M * l.top * (2.0 * D + 8.0 * l.expert_ff + 2.0 * l.expert_ff + 4.0 * D))
+        add("dense", 2.0 * M * wd, 2.0 * wd + act)
+    return {k: tuple(v) for k, v in cls.items()}
+
+
 def family_model(cfg, M, kv_len, nseq, peaks):
     """algorithmic FLOPs and bytes of one forward of M tokens (nseq sequences, kv_len keys each) per kernel class"""
     import math
     L = cfg.num_hidden_layers
-    if getattr(cfg, "architecture", None) in ("Rivetar", "Mavipel", "Lukopel", "Dikopel"):
+    if getattr(cfg, "architecture", None) in ("Rivetar", "Mavipel", "Lukopel", "Dikopel", "Nobonex"):
         L = 1           # these models already sum over the layer executions
         cls = {"Rivetar": rivetar_model, "Mavipel": mavipel_model, "Lukopel": lukopel_model,
-               "Dikopel": dikopel_model}[cfg.architecture](cfg, M, kv_len, nseq)
+               "Dikopel": dikopel_model, "Nobonex": nobonex_model}[cfg.architecture](cfg, M, kv_len, nseq)
         head = (2.0 * nseq * cfg.vocab_size * cfg.width, 2.0 * cfg.vocab_size * cfg.width)
     elif getattr(cfg, "architecture", None) == "Mezilix":
         l, D = cfg.layers[0], cfg.width
@@ -909,18 +951,19 @@ def family_model(cfg, M, kv_len, nseq, peaks):
 
 
 def run_family(args):
-    """--family mezilix | rivetar | mavipel | lukopel | dikopel: prefill and decode throughput of that family's engine at layer sizes
+    """--family mezilix | rivetar | mavipel | lukopel | dikopel | nobonex: prefill and decode throughput of that family's engine at layer sizes
     of real models, beside the Qwen2 engine at the same width, depth, head count and active weights per layer (Mavipel:
-    beside the Rivetar engine, Lukopel and Dikopel: beside the Mavipel engine, at the same width, depth and head count); random
-    weights, synthetic tokens.
+    beside the Rivetar engine, Lukopel and Dikopel: beside the Mavipel engine, Nobonex: beside the Dikopel engine, at the same
+    width, depth and head count); random weights, synthetic tokens.
     Per kernel class: device time (CUDA events around every launch) against its floor = max(FLOPs / measured cuBLAS bf16
     rate, bytes / measured copy bandwidth).  Prints one JSON object; the default workload of this file is untouched."""
     import torch
     import asd_b200  # noqa: F401
-    from asd_b200.engine import DikopelEngine, LukopelEngine, MavipelEngine, MezilixEngine, QwenEngine, RivetarEngine
+    from asd_b200.engine import (DikopelEngine, LukopelEngine, MavipelEngine, MezilixEngine, NobonexEngine, QwenEngine,
+                                 RivetarEngine)
     from asd_b200.models import registry
     engines = {"mezilix": MezilixEngine, "rivetar": RivetarEngine, "mavipel": MavipelEngine, "lukopel": LukopelEngine,
-               "dikopel": DikopelEngine,
+               "dikopel": DikopelEngine, "nobonex": NobonexEngine,
                "qwen2": QwenEngine}
     path = os.path.join(ROOT, "MEASURED_PEAKS.json")
     peaks = json.load(open(path)) if os.path.exists(path) else {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0}
@@ -1021,7 +1064,7 @@ def main():
     ap.add_argument("--no-fuse-norm", action="store_true", help="separate add+RMSNorm kernels instead of the fused epilogues")
     ap.add_argument("--nccl-only", action="store_true", help="TP boundaries through ncclAllReduce instead of the fused kernel")
     ap.add_argument("--opt", action="append", help="engine option name=value (e.g. pdl=0, attn_impl=0)")
-    ap.add_argument("--family", default=None, choices=["mezilix", "rivetar", "mavipel", "lukopel", "dikopel"],
+    ap.add_argument("--family", default=None, choices=["mezilix", "rivetar", "mavipel", "lukopel", "dikopel", "nobonex"],
                     help="instead of the default workload: prefill / decode throughput of this model family beside its closest "
                          "existing family at equal size")
     args = ap.parse_args()
