@@ -25,7 +25,7 @@
 // active warps).  Long contexts are split over the KV length (flash decoding) with the same ticket merge as
 // attention.cu.
 //
-// The reference has no attention code (vLLM does it: /root/reference/src/serving/real_model_pipeline.py:98-108);
+// The reference has no attention code (vLLM does it: src/serving/real_model_pipeline.py:98-108);
 // semantics are HF Qwen2 GQA attention with softmax scale 1/sqrt(head_dim), causal among the new positions.
 #include <cuda.h>
 #include <cuda_bf16.h>

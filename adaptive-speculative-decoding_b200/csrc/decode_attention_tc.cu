@@ -152,6 +152,11 @@ __global__ void __launch_bounds__(NT) decode_tc_kernel(MixArgs a) {
         uint32_t ph[4], pl[4];
         if (SOFT) {
 #pragma unroll
+            for (int n = 0; n < 2; ++n)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) s[n][e] *= a.d.scale;
+            if (MODE == D_SOFTMAX_CAP) cap_scores(s, a.d.softcap, icap);
+#pragma unroll
             for (int x = 0; x < 2; ++x) {
                 float mx = -INFINITY;
 #pragma unroll
@@ -159,22 +164,20 @@ __global__ void __launch_bounds__(NT) decode_tc_kernel(MixArgs a) {
 #pragma unroll
                     for (int e = 0; e < 2; ++e) {
                         const int j = j0 + n * 8 + 2 * t4 + e;
-                        float v = s[n][2 * x + e] * a.d.scale;
-                        if (MODE == D_SOFTMAX_CAP) v = cap_score(v, a.d.softcap, icap);
-                        v = j <= posr[x] && j >= lor[x] ? v : -INFINITY;
+                        const float v = j <= posr[x] && j >= lor[x] ? s[n][2 * x + e] : -INFINITY;
                         s[n][2 * x + e] = v;
                         mx = fmaxf(mx, v);
                     }
                 mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
                 mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
                 const float mnew = fmaxf(mrun[x], mx), ref = mnew > -INFINITY ? mnew : 0.f;
-                const float keep = expf(mrun[x] - ref);
+                const float keep = __expf(mrun[x] - ref);
                 float sum = 0.f;           // this thread's part of the row's sum; the quad's parts are added at the end
 #pragma unroll
                 for (int n = 0; n < 2; ++n)
 #pragma unroll
                     for (int e = 0; e < 2; ++e) {
-                        s[n][2 * x + e] = expf(s[n][2 * x + e] - ref);
+                        s[n][2 * x + e] = __expf(s[n][2 * x + e] - ref);
                         sum += s[n][2 * x + e];
                     }
                 lrun[x] = fmaf(lrun[x], keep, sum);

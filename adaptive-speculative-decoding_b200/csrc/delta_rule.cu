@@ -134,7 +134,61 @@ __global__ void short_conv_kernel(SeqIndex ix, const float* in, long long ld, co
     }
 }
 
-// the last ring_n new positions of every sequence leave their inputs behind (runs after short_conv_kernel has read)
+// Prompts: a thread takes four consecutive channels down a run of consecutive rows and keeps the N - 1 inputs before its row
+// in registers, so an input is read once per run.  Where a row is not the position after the row above, its window is read
+// anew: from the rows above while they belong to the sequence, else from the ring, zeros before position 0.
+constexpr int CONV_RUN = 16;
+template <int MODE, int N>
+__global__ void __launch_bounds__(128) short_conv_run_kernel(SeqIndex ix, const float* in, long long ld, const float* taps, int C,
+                                                             const float* ring, int ring_n, void* out, int of32, const float* bias) {
+    const int c = (blockIdx.y * blockDim.x + threadIdx.x) * 4;
+    if (c >= C) return;
+    const int m0 = blockIdx.x * CONV_RUN, m1 = min(ix.M, m0 + CONV_RUN);
+    float tap[4][N], b[4] = {0.f, 0.f, 0.f, 0.f}, win[N][4];     // win[j]: the input N - 1 - j positions back
+#pragma unroll
+    for (int e = 0; e < 4; ++e)
+#pragma unroll
+        for (int j = 0; j < N; ++j) tap[e][j] = __ldg(taps + (long long)(c + e) * N + j);
+    if (bias) ldx4(bias, c, 1, b);
+    int slot = -1, next = -1;
+    for (int m = m0; m < m1; ++m) {
+        const int pos = ix.positions[m], sl = ix.token_slot[m];
+        if (sl == slot && pos == next) {
+#pragma unroll
+            for (int j = 0; j + 1 < N; ++j)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) win[j][e] = win[j + 1][e];
+        } else {
+            bool same = true;                                     // rows above still belong to this sequence
+#pragma unroll
+            for (int back = 1; back < N; ++back) {
+                float(&v)[4] = win[N - 1 - back];
+                const int p = pos - back, r = m - back;
+                same = same && r >= 0 && ix.token_slot[r] == sl && ix.positions[r] == p;
+                if (p < 0)
+                    v[0] = v[1] = v[2] = v[3] = 0.f;
+                else if (same)
+                    ldx4(in, (long long)r * ld + c, 1, v);
+                else
+                    ldx4(ring, ((long long)sl * ring_n + p % ring_n) * C + c, 1, v);
+            }
+        }
+        slot = sl, next = pos + 1;
+        ldx4(in, (long long)m * ld + c, 1, win[N - 1]);
+        float o[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            float acc = 0.f;
+#pragma unroll
+            for (int j = 0; j < N; ++j) acc = fmaf(tap[e][j], win[j][e], acc);
+            acc += b[e];
+            o[e] = MODE == CONV_RESIDUAL ? win[N - 1][e] + acc : (MODE == CONV_PLAIN ? acc : acc / (1.f + expf(-acc)));
+        }
+        stx4(out, (long long)m * C + c, of32, o);
+    }
+}
+
+// the last ring_n new positions of every sequence leave their inputs behind (runs after the convolution has read)
 __global__ void conv_commit_kernel(SeqIndex ix, const int* cu_q, const float* in, long long ld, int C, float* ring,
                                    int ring_n) {
     const int seq = blockIdx.x;
@@ -142,8 +196,8 @@ __global__ void conv_commit_kernel(SeqIndex ix, const int* cu_q, const float* in
     for (int m = t0 + blockIdx.y; m < t1; m += gridDim.y) {
         const int pos = ix.positions[m], slot = ix.token_slot[m];
         float* dst = ring + ((long long)slot * ring_n + pos % ring_n) * C;
-#pragma unroll 8
-        for (int c = threadIdx.x; c < C; c += blockDim.x) dst[c] = __ldg(in + (long long)m * ld + c);
+#pragma unroll 4
+        for (int c = blockIdx.z * blockDim.x + threadIdx.x; c < C; c += gridDim.z * blockDim.x) dst[c] = __ldg(in + (long long)m * ld + c);
     }
 }
 
@@ -677,6 +731,25 @@ int launch_carried_conv(const SeqIndex& ix, const int* cu_q, int nseq, int max_q
     dim3 grid(ix.M, (C + 4 * threads - 1) / (4 * threads));
     if (grid.y > 65535) return set_error("short_conv: too many channels");
     const int rn = ring_n > 0 ? ring_n : 1;
+    uintptr_t at = 0;
+    for (const void* p : {(const void*)in, (const void*)ring, (const void*)out, (const void*)bias}) at |= reinterpret_cast<uintptr_t>(p);
+    if (max_qlen >= CONV_RUN && n_taps >= 2 && n_taps <= 5 && C % 4 == 0 && ld % 4 == 0 && (at & 15) == 0) {
+        const dim3 rgrid((ix.M + CONV_RUN - 1) / CONV_RUN, (C / 4 + 127) / 128);
+        auto runs = [&](auto kernel) { kernel<<<rgrid, 128, 0, stream>>>(ix, in, ld, taps, C, ring, rn, out, of32, bias); };
+#define ASD_CONV_N(MODE)                                                                                                       \
+    n_taps == 2 ? runs(short_conv_run_kernel<MODE, 2>) : n_taps == 3 ? runs(short_conv_run_kernel<MODE, 3>)                     \
+                : n_taps == 4 ? runs(short_conv_run_kernel<MODE, 4>) : runs(short_conv_run_kernel<MODE, 5>)
+        if (mode == CONV_RESIDUAL)
+            ASD_CONV_N(CONV_RESIDUAL);
+        else if (mode == CONV_PLAIN)
+            ASD_CONV_N(CONV_PLAIN);
+        else
+            ASD_CONV_N(CONV_SILU);
+#undef ASD_CONV_N
+        count_launch(1);
+        ASD_CUDA(cudaGetLastError());
+        return launch_conv_commit(ix, cu_q, nseq, in, ld, C, ring, ring_n, stream);
+    }
     auto run = [&](auto kernel) {
         kernel<<<grid, threads, 0, stream>>>(ix, in, ld, taps, n_taps, C, ring, single ? ring : nullptr, rn, out, of32, bias);
     };
@@ -695,8 +768,9 @@ int launch_carried_conv(const SeqIndex& ix, const int* cu_q, int nseq, int max_q
 int launch_conv_commit(const SeqIndex& ix, const int* cu_q, int nseq, const float* in, long long ld, int C, float* ring,
                        int ring_n, cudaStream_t stream) {
     if (ix.M <= 0 || nseq <= 0 || ring_n <= 0 || C <= 0) return 0;
-    dim3 grid(nseq, ring_n < 16 ? ring_n : 16);
-    conv_commit_kernel<<<grid, C >= 1024 ? 256 : 128, 0, stream>>>(ix, cu_q, in, ld, C, ring, ring_n);
+    const int threads = C >= 1024 ? 256 : 128;
+    dim3 grid(nseq, ring_n < 16 ? ring_n : 16, nseq < 64 ? (C + 4 * threads - 1) / (4 * threads) : 1);
+    conv_commit_kernel<<<grid, threads, 0, stream>>>(ix, cu_q, in, ld, C, ring, ring_n);
     count_launch(1);
     ASD_CUDA(cudaGetLastError());
     return 0;

@@ -4,7 +4,7 @@
 // the caller's stream with no host synchronisation (CUDA-graph capturable).
 //
 // This is the slot the reference fills with vllm.LLM(...).generate
-// (/root/reference/src/serving/real_model_pipeline.py:98-108,135; Stage listing in
+// (src/serving/real_model_pipeline.py:98-108,135; Stage listing in
 // docs/guides/RESEARCH_PROTOCOL.md:233-304).  Tensor parallelism mirrors what vLLM does for the
 // reference's `tensor_parallel_size` (configs/qwen3_models.yaml:10,22,34,46): column-parallel
 // QKV / gate|up, row-parallel O / down, one all-reduce after each row-parallel GEMM.

@@ -29,7 +29,7 @@
 // global spin is bounded and reports through PersistLaunch::error.
 //
 // Stands behind Stage.generate's model forward, which the reference delegates to vLLM
-// (/root/reference/src/serving/real_model_pipeline.py:98-108,135).
+// (src/serving/real_model_pipeline.py:98-108,135).
 #include <cuda.h>
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>

@@ -26,7 +26,7 @@
 // Programmatic dependent launch: weight stages are issued before griddepcontrol.wait, activations after it.
 //
 // Stands behind Stage.generate's model forward, which the reference delegates to vLLM
-// (/root/reference/src/serving/real_model_pipeline.py:98-108,135).
+// (src/serving/real_model_pipeline.py:98-108,135).
 #include <cuda.h>
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>

@@ -19,7 +19,7 @@
 // interleaved 64 gate / 64 up rows per 128-row tile (same layout as gemm.cu).
 //
 // Stands behind Stage.generate's model forward, which the reference delegates to vLLM
-// (/root/reference/src/serving/real_model_pipeline.py:98-108,135).
+// (src/serving/real_model_pipeline.py:98-108,135).
 #include <cuda.h>
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>

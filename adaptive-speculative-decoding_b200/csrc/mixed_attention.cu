@@ -676,9 +676,24 @@ __global__ void __launch_bounds__(NT) mix_dec_apply_kernel(MixArgs a) {
     }
 }
 
-// A warp per query, key and value head in turn.  Dynamic shared memory: the row (n floats), the heads' sums of squares,
+template <int V>
+__device__ __forceinline__ void ldv(const float* p, float (&v)[V]) {
+    if constexpr (V == 4)
+        ldx4(p, 0, 1, v);
+    else
+        v[0] = *p;
+}
+template <int V, typename T>
+__device__ __forceinline__ void stv(T* p, const float (&v)[V]) {
+    if constexpr (V == 4)
+        stx4(p, 0, sizeof(T) == 4, v);
+    else
+        stf(p, v[0]);
+}
+
+// A warp per query, key and value head in turn, V consecutive elements a lane.  Dynamic shared memory: the row (n floats), the heads' sums of squares,
 // cos and sin of the token's angles.
-template <typename T>
+template <typename T, int V>
 __global__ void mix_post_kernel(SeqIndex ix, float* qkv, long long ld, MixDims d, MixPost p, PagedRows cache) {
     extern __shared__ float sm[];
     const int H = d.heads, G = d.kv_heads, dk = d.dk, dv = d.dv;
@@ -700,10 +715,17 @@ __global__ void mix_post_kernel(SeqIndex ix, float* qkv, long long ld, MixDims d
     for (int u = warp; u < units; u += nw) {
         const int beg = u < ku ? u * dk : nq + nk + (u - ku) * dv, len = u < ku ? dk : dv;
         float ss = 0.f;
-        for (int i = lane; i < len; i += 32) {
-            const float v = src[beg + i] + (p.bias ? p.bias[beg + i] : 0.f);
-            row[beg + i] = v;
-            ss = fmaf(v, v, ss);
+        for (int i = lane * V; i < len; i += 32 * V) {
+            float v[V], b[V];
+            ldv<V>(src + beg + i, v);
+            if (p.bias) {
+                ldv<V>(p.bias + beg + i, b);
+#pragma unroll
+                for (int e = 0; e < V; ++e) v[e] += b[e];
+            }
+            stv<V>(row + beg + i, v);
+#pragma unroll
+            for (int e = 0; e < V; ++e) ss = fmaf(v[e], v[e], ss);
         }
         ss = warp_sum(ss);
         if (lane == 0) ss_of[u] = ss;
@@ -729,7 +751,13 @@ __global__ void mix_post_kernel(SeqIndex ix, float* qkv, long long ld, MixDims d
         if (u >= ku) {                                     // a value head
             const int g = u - ku;
             const float f = p.v_unit ? 1.f / sqrtf(ss_of[u] / (float)dv + p.eps) : 1.f;
-            for (int i = lane; i < dv; i += 32) stf(dst + G * dk + g * dv + i, row[nq + nk + g * dv + i] * f);
+            for (int i = lane * V; i < dv; i += 32 * V) {
+                float v[V];
+                ldv<V>(row + nq + nk + g * dv + i, v);
+#pragma unroll
+                for (int e = 0; e < V; ++e) v[e] *= f;
+                stv<V>(dst + G * dk + g * dv + i, v);
+            }
             continue;
         }
         const bool is_q = u < H;
@@ -742,19 +770,31 @@ __global__ void mix_post_kernel(SeqIndex ix, float* qkv, long long ld, MixDims d
         }
         const float* r = row + u * dk;
         const float* w = nw_ ? nw_ + (p.norm_whole ? (is_q ? u : u - H) * dk : 0) : nullptr;
-        for (int i = lane; i < dk; i += 32) {
-            float v = r[i] * f * (w ? w[i] : 1.f);
-            if (i < p.rot_dims) {
-                const int j = p.rot_interleaved ? i ^ 1 : (i < half ? i + half : i - half);
-                const int pair = p.rot_interleaved ? i >> 1 : (i < half ? i : j);
-                const float o = r[j] * f * (w ? w[j] : 1.f);
-                v = fmaf(v, cs[pair], i < j ? -o * cs[half + pair] : o * cs[half + pair]);
-            }
+        const float unit = p.v_from_k && p.v_unit ? 1.f / sqrtf(ss_of[u] / (float)dk + p.eps) : 1.f;
+        for (int i = lane * V; i < dk; i += 32 * V) {
+            float raw[V], v[V];
+            ldv<V>(r + i, raw);
+#pragma unroll
+            for (int e = 0; e < V; ++e) v[e] = raw[e] * f * (w ? w[i + e] : 1.f);
+            if (i < p.rot_dims)
+#pragma unroll
+                for (int e = 0; e < V; ++e) {
+                    const int d = i + e;
+                    if (d >= p.rot_dims) break;
+                    const int j = p.rot_interleaved ? d ^ 1 : (d < half ? d + half : d - half);
+                    const int pair = p.rot_interleaved ? d >> 1 : min(d, j);
+                    const float o = r[j] * f * (w ? w[j] : 1.f);
+                    v[e] = fmaf(v[e], cs[pair], d < j ? -o * cs[half + pair] : o * cs[half + pair]);
+                }
             if (is_q) {
-                src[u * dk + i] = v;
+                stv<V>(src + u * dk + i, v);
             } else {
-                stf(dst + (u - H) * dk + i, v);
-                if (p.v_from_k) stf(dst + G * dk + (u - H) * dv + i, r[i] * (p.v_unit ? 1.f / sqrtf(ss_of[u] / (float)dk + p.eps) : 1.f));
+                stv<V>(dst + (u - H) * dk + i, v);
+                if (p.v_from_k) {
+#pragma unroll
+                    for (int e = 0; e < V; ++e) raw[e] *= unit;
+                    stv<V>(dst + G * dk + (u - H) * dv + i, raw);
+                }
             }
         }
     }
@@ -795,13 +835,19 @@ int launch_mix_post(const SeqIndex& ix, float* qkv, long long ld, const MixDims&
     if (smem > 200 * 1024) return set_error("mix_post: a row of %d values does not fit shared memory", n);
     static PerDeviceOnce once;
     if (once.need()) {
-        ASD_CUDA(cudaFuncSetAttribute(mix_post_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
-        ASD_CUDA(cudaFuncSetAttribute(mix_post_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
+        ASD_CUDA(cudaFuncSetAttribute(mix_post_kernel<float, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
+        ASD_CUDA(cudaFuncSetAttribute(mix_post_kernel<float, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
+        ASD_CUDA(cudaFuncSetAttribute(mix_post_kernel<__nv_bfloat16, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
+        ASD_CUDA(cudaFuncSetAttribute(mix_post_kernel<__nv_bfloat16, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
     }
+    const uintptr_t at = reinterpret_cast<uintptr_t>(qkv) | reinterpret_cast<uintptr_t>(p.bias) |
+                         (p.q_only ? 0 : reinterpret_cast<uintptr_t>(cache.pool));
+    const bool four = d.dk % 4 == 0 && d.dv % 4 == 0 && ld % 4 == 0 && (at & 15) == 0;
+    auto run = [&](auto kernel) { kernel<<<ix.M, threads, smem, stream>>>(ix, qkv, ld, d, p, cache); };
     if (cache.f32)
-        mix_post_kernel<float><<<ix.M, threads, smem, stream>>>(ix, qkv, ld, d, p, cache);
+        four ? run(mix_post_kernel<float, 4>) : run(mix_post_kernel<float, 1>);
     else
-        mix_post_kernel<__nv_bfloat16><<<ix.M, threads, smem, stream>>>(ix, qkv, ld, d, p, cache);
+        four ? run(mix_post_kernel<__nv_bfloat16, 4>) : run(mix_post_kernel<__nv_bfloat16, 1>);
     count_launch(1);
     ASD_CUDA(cudaGetLastError());
     return 0;

@@ -37,13 +37,25 @@ __device__ __forceinline__ float mix_gate(const MixArgs& a, long long m, int h, 
     return 1.f / (1.f + expf(-a.gate[m * a.ldg + (a.d.gate_per_value ? h * a.d.dv + col : h)]));
 }
 
-// cap * tanh(v / cap): the Taylor series of tanh to the seventh power below 1/4, 1 - 2 / (1 + e^(2a)) above; relative error
-// below 1e-6
-__device__ __forceinline__ float cap_score(float v, float cap, float icap) {
-    const float a = fabsf(v) * icap, a2 = a * a;
-    const float big = 1.f - __fdividef(2.f, 1.f + __expf(2.f * a));
-    const float small = a * fmaf(a2, fmaf(a2, fmaf(a2, -17.f / 315.f, 2.f / 15.f), -1.f / 3.f), 1.f);
-    return copysignf(cap * (a < 0.25f ? small : big), v);
+// cap * tanh(v / cap) of a warp's scores: the Taylor series of tanh to the seventh power where all of them lie below a quarter
+// of the cap, else 1 - 2 / (1 + e^(2a)) for those beyond it; relative error below 1e-6
+template <int N>
+__device__ __forceinline__ void cap_scores(float (&s)[N][4], float cap, float icap) {
+    float top = 0.f;
+#pragma unroll
+    for (int n = 0; n < N; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) top = fmaxf(top, fabsf(s[n][e]));
+    const bool beyond = __any_sync(0xffffffffu, !(top * icap < 0.25f));
+#pragma unroll
+    for (int n = 0; n < N; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const float v = s[n][e], a = v * icap, a2 = a * a;
+            float r = v * fmaf(a2, fmaf(a2, fmaf(a2, -17.f / 315.f, 2.f / 15.f), -1.f / 3.f), 1.f);
+            if (beyond && fabsf(a) >= 0.25f) r = copysignf(cap * (1.f - __fdividef(2.f, 1.f + __expf(2.f * fabsf(a)))), v);
+            s[n][e] = r;
+        }
 }
 
 // Prompts and portions of a bf16 engine on the tensor cores (mma.sync, fp32 operands as two bf16 terms).  Returns 1 if

@@ -109,7 +109,7 @@ __global__ void __launch_bounds__(NT) mix_tc_kernel(MixArgs a) {
     const int M = a.ix.M;
     const float icap = CAP ? 1.f / a.d.softcap : 0.f;
     const int p0 = a.ix.positions[q_beg], p1 = p0 + nq - 1;
-    const int kmin = chunk > 0 ? (p0 / chunk) * chunk : 0;
+    const int kmin = chunk > 0 ? (p0 / chunk) * chunk : 0, lo_last = chunk > 0 ? (p1 / chunk) * chunk : 0;
     const int ntile = (p1 - kmin) / KT + 1;
     const int per = (ntile + a.shares - 1) / a.shares;
     const int t0 = share * per, t1 = min(ntile, t0 + per);
@@ -244,24 +244,36 @@ __global__ void __launch_bounds__(NT) mix_tc_kernel(MixArgs a) {
 #pragma unroll
             for (int n = 0; n < KT / 8; ++n)
 #pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    const int x = e >> 1, col = n * 8 + 2 * t + (e & 1), j = kb + col;
-                    const bool ok = okx[x] && col < nk && j <= posx[x] && j >= lox[x];
-                    float v = s[n][e] * a.d.scale;
-                    if (CAP) v = cap_score(v, a.d.softcap, icap);
-                    if (a.dist_bias && ok) v += a.dist_bias[(long long)min(posx[x] - j, a.far) * H + hx[x]];
-                    if (MODE == SIGMOID) {
-                        s[n][e] = ok ? __fdividef(1.f, 1.f + __expf(-(v + hbx[x]))) : 0.f;
-                        continue;
+                for (int e = 0; e < 4; ++e) s[n][e] *= a.d.scale;
+            if (CAP) cap_scores(s, a.d.softcap, icap);
+            if (ONE && !a.dist_bias && nk == KT && kb + KT - 1 <= p0 && kb >= lo_last) {
+                // every row sees the whole tile (rows beyond the portion compute what nobody stores)
+#pragma unroll
+                for (int n = 0; n < KT / 8; ++n)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) tmax[e >> 1] = fmaxf(tmax[e >> 1], s[n][e]);
+            } else {
+#pragma unroll
+                for (int n = 0; n < KT / 8; ++n)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        const int x = e >> 1, col = n * 8 + 2 * t + (e & 1), j = kb + col;
+                        const bool ok = okx[x] && col < nk && j <= posx[x] && j >= lox[x];
+                        float v = s[n][e];
+                        if (a.dist_bias && ok) v += a.dist_bias[(long long)min(posx[x] - j, a.far) * H + hx[x]];
+                        if (MODE == SIGMOID) {
+                            s[n][e] = ok ? __fdividef(1.f, 1.f + __expf(-(v + hbx[x]))) : 0.f;
+                            continue;
+                        }
+                        v = ok ? v : -INFINITY;
+                        if (!APPLY || ONE) {
+                            s[n][e] = v;
+                            tmax[x] = fmaxf(tmax[x], v);
+                        } else {
+                            s[n][e] = ok ? expf(v - Mx[x]) * iLx[x] : 0.f;
+                        }
                     }
-                    v = ok ? v : -INFINITY;
-                    if (!APPLY || ONE) {
-                        s[n][e] = v;
-                        tmax[x] = fmaxf(tmax[x], v);
-                    } else {
-                        s[n][e] = ok ? expf(v - Mx[x]) * iLx[x] : 0.f;
-                    }
-                }
+            }
             if (!APPLY) {
 #pragma unroll
                 for (int x = 0; x < 2; ++x) {
@@ -289,20 +301,19 @@ __global__ void __launch_bounds__(NT) mix_tc_kernel(MixArgs a) {
                 for (int x = 0; x < 2; ++x) {
                     tmax[x] = fmaxf(tmax[x], __shfl_xor_sync(0xffffffffu, tmax[x], 1));
                     tmax[x] = fmaxf(tmax[x], __shfl_xor_sync(0xffffffffu, tmax[x], 2));
-                    const float mnew = fmaxf(mrun[x], tmax[x]);
-                    const float keep = (mrun[x] > -INFINITY && mnew > -INFINITY) ? expf(mrun[x] - mnew) : 0.f;
+                    const float mnew = fmaxf(mrun[x], tmax[x]), ref = mnew > -INFINITY ? mnew : 0.f;
+                    const float keep = __expf(mrun[x] - ref);
                     float sum = 0.f;      // this thread's part of the row's sum; the quad's parts are added at the end
 #pragma unroll
                     for (int n = 0; n < KT / 8; ++n) {
-                        const float w0 = s[n][2 * x] > -INFINITY ? expf(s[n][2 * x] - mnew) : 0.f;
-                        const float w1 = s[n][2 * x + 1] > -INFINITY ? expf(s[n][2 * x + 1] - mnew) : 0.f;
-                        s[n][2 * x] = w0, s[n][2 * x + 1] = w1;
-                        sum += w0 + w1;
+                        s[n][2 * x] = __expf(s[n][2 * x] - ref), s[n][2 * x + 1] = __expf(s[n][2 * x + 1] - ref);
+                        sum += s[n][2 * x] + s[n][2 * x + 1];
                     }
                     lrun[x] = lrun[x] * keep + sum;
                     mrun[x] = mnew;
+                    if (__any_sync(0xffffffffu, keep != 1.f))
 #pragma unroll
-                    for (int n = 0; n < NDV; ++n) O[n][2 * x] *= keep, O[n][2 * x + 1] *= keep;
+                        for (int n = 0; n < NDV; ++n) O[n][2 * x] *= keep, O[n][2 * x + 1] *= keep;
                 }
             } else if (TALK) {
 #pragma unroll

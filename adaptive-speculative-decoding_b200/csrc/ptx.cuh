@@ -1,6 +1,5 @@
 // Thin inline-PTX wrappers for sm_100a: mbarrier, bulk/TMA copies, clusters, tcgen05/TMEM.
-// No CUTLASS dependency; bit layouts follow the PTX ISA (tcgen05 descriptors) as documented in
-// /opt/skills/guides/blackwell_cuda_programming.md.
+// No CUTLASS dependency; bit layouts follow the PTX ISA (tcgen05 descriptors).
 #pragma once
 #include <cuda_runtime.h>
 #include <stdint.h>

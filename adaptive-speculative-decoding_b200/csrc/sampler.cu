@@ -24,7 +24,7 @@
 // Inside a chunk, local element u lives in lane (u / 4) mod 256 = thread, visited in increasing u.
 //
 // Replaces (reference): per-token softmax + log(probs[token]) with a host sync per token,
-// /root/reference/src/training/generate_training_data.py:128-134, and the logprob feature
+// src/training/generate_training_data.py:128-134, and the logprob feature
 // reductions of docs/guides/RESEARCH_PROTOCOL.md:379-398.  The accept/resample rule itself has no
 // reference implementation.
 #include <cuda_runtime.h>

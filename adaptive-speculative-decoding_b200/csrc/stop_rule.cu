@@ -1,5 +1,5 @@
 // Cascade stop rule: backward-induction DP of the reference's optimal_stopping_rule
-// (/root/reference/src/algorithms/dp_solver.py:12-71) and the Beta-posterior shrinkage
+// (src/algorithms/dp_solver.py:12-71) and the Beta-posterior shrinkage
 // bayesian_adjustment (:106-130), evaluated for a batch of requests on the device so the
 // stop decision needs no logits/feature round trip, plus the same arithmetic as a host
 // function for the scalar Python API (policy seam 3, pipeline.py:236-238,251-256).
@@ -96,7 +96,7 @@ __global__ void stop_rule_kernel(const double* __restrict__ p, const double* __r
 // DP, and emits (acceptance probability, stop?, k*).  The host only reads those three numbers per request: no logits,
 // no per-token features and no MLP on the host.  Mirrors FeatureExtractor.extract + QualityPredictor.predict +
 // bayesian_adjustment + optimal_stopping_rule as chained by the reference's loop
-// (/root/reference/src/serving/pipeline.py:225-256; listing docs/guides/RESEARCH_PROTOCOL.md:366-409).
+// (src/serving/pipeline.py:225-256; listing docs/guides/RESEARCH_PROTOCOL.md:366-409).
 constexpr int kHidden = 128;
 
 struct CascadeArgs {

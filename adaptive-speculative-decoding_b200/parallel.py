@@ -4,7 +4,7 @@ NCCL communicator (created through ctypes on the NCCL library torch already load
 the two row-parallel boundaries of every layer.
 
 Mirrors the reference's ``tensor_parallel_size`` knob, which it passes to vLLM
-(/root/reference/src/serving/real_model_pipeline.py:100; configs/qwen3_models.yaml:10,22,34,46)."""
+(src/serving/real_model_pipeline.py:100; configs/qwen3_models.yaml:10,22,34,46)."""
 from __future__ import annotations
 
 import ctypes

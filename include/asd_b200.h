@@ -2,7 +2,7 @@
  * asd_b200.h - C ABI of libasd_b200.so, the B200-native (sm_100a) draft-then-verify hot path
  * behind the adaptive-speculative-decoding Python API.
  *
- * The reference (sa2shun/adaptive-speculative-decoding, /root/reference) is 100 % Python and has
+ * The reference (sa2shun/adaptive-speculative-decoding) is 100 % Python and has
  * NO FFI for this path: its engine seam is duck-typed Python that delegates to vLLM
  * (src/serving/real_model_pipeline.py:98-108,135; docs/guides/RESEARCH_PROTOCOL.md:233-304).
  * Each entry point below therefore cites the Python interface it stands behind; the ctypes

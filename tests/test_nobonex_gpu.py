@@ -454,6 +454,29 @@ def test_batched_single_token_and_few_token_steps():
         close(eng)
 
 
+def test_prompt_beside_single_tokens_and_short_portions():
+    """one step brings a long prompt, a long portion that continues a state, single tokens and two tokens; the step after
+    it single tokens of all four"""
+    w = O.random_model(SMALL, seed=32)
+    seqs = [tokens(n, 120, 50 + n) for n in (90, 130, 41, 30)]
+    refs = [oracle(SMALL, w, s) for s in seqs]
+    for dtype in (torch.float32, torch.bfloat16):
+        eng = make_engine(SMALL, w, max_tokens=256, dtype=dtype, page_size=8)
+        slots = [eng.open_sequence() for _ in seqs]
+        for sl, s in zip(slots, seqs):
+            eng.reserve(sl, len(s))
+        eng.forward_ragged([(slots[1], 0, seqs[1][:50], []), (slots[2], 0, seqs[2][:38], []), (slots[3], 0, seqs[3][:25], [])])
+        at = [0, 50, 38, 25]
+        for sizes in ((85, 75, 1, 2), (1, 1, 1, 1), (4, 4, 1, 2)):
+            out = eng.forward_ragged([(sl, a, s[a:a + n], list(range(n))) for sl, s, a, n in zip(slots, seqs, at, sizes)])
+            o = 0
+            for i, n in enumerate(sizes):
+                g, r = out[o:o + n], refs[i][at[i]:at[i] + n]
+                o, at[i] = o + n, at[i] + n
+                assert (rel_err(g, r)[1] < 2e-4) if dtype == torch.float32 else (rel_err(g, r)[0] < 8e-2), (i, sizes)
+        close(eng)
+
+
 def test_pages_slots_and_state_freed_and_used_again():
     """a pool with room for one request at a time: the second request gets the first one's slot, pages, carried inputs
     and states with the old contents still in them"""
