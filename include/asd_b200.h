@@ -631,8 +631,8 @@ ASD_API int asd_dikopel_device_error(asd_dikopel_engine_t* e);
  *           causal softmax attention over scale * q . k;
  *   type 1  scalar-decay state space recurrence: projection [z | x | B | C | dt] with z, x heads * vdim, B, C groups * state,
  *           dt heads values; x, B, C pass a causal convolution with bias and silu; dt <- softplus(dt + dt_bias);
- *           S <- exp(-exp(a_log) dt) S + dt B x^T, y = S^T C + skip x per head; y * silu(z) is RMS-normed in norm_groups equal
- *           parts, times out_norm;
+ *           S <- exp(-exp(a_log) dt) S + dt B x^T, y = S^T C + skip x per head; then u = y * silu(z), each of norm_groups
+ *           consecutive slices of u over its own rms(u), * out_norm;
  *   type 2  chunked attention (heads, kv_heads, dim, vdim): biased projections, RMS norm per head, rotation in pairs
  *           (i, i + rot_dims/2), scores scale * q . k capped as softcap * tanh(. / softcap) (0: not), position i sees j <= i
  *           with i / chunk == j / chunk (chunk 0: every j <= i), softmax; the result times sigmoid of a projection of the

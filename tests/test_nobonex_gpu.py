@@ -237,7 +237,7 @@ def test_many_tokens_take_the_other_routing_kernel():
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16], ids=["fp32", "bf16"])
 @pytest.mark.parametrize("heads,kv,dim,taps,rot", [(6, 2, 24, 3, 12), (4, 4, 32, 1, 32), (8, 1, 64, 2, 0), (20, 4, 16, 7, 4), (12, 1, 40, 4, 40),
-                                                   (5, 5, 10, 5, 6), (2, 1, 136, 3, 64), (34, 1, 16, 4, 8), (3, 1, 200, 2, 2), (24, 2, 128, 4, 96)])
+                                                   (5, 5, 10, 5, 6), (2, 1, 136, 3, 64), (34, 1, 16, 4, 8), (3, 1, 200, 2, 2), (24, 2, 128, 4, 96), (2, 1, 256, 4, 64)])
 def test_convolved_attention_alone(heads, kv, dim, taps, rot, dtype):
     """every kernel: prompts, portions of a few tokens, single tokens; sizes that fill a load and that do not; more than
     eight and sixteen query heads per key head; a large oldest tap makes a lost or misplaced carried row show"""
@@ -264,7 +264,7 @@ def test_convolved_attention_alone(heads, kv, dim, taps, rot, dtype):
 @pytest.mark.parametrize("heads,kv,dim,vdim,chunk,cap,rot,factor", [
     (4, 2, 32, 24, 24, 20.0, 16, 4.0), (4, 4, 32, 64, 64, 2.0, 32, 1.0), (8, 1, 64, 128, 33, 50.0, 8, 2.0), (20, 4, 16, 16, 200, 1.0, 4, 0.0),
     (12, 1, 40, 24, 1000, 5.0, 40, 40.0), (5, 5, 10, 6, 7, 3.0, 6, 8.0), (2, 1, 136, 200, 1, 30.0, 64, 1.5), (34, 1, 16, 16, 17, 10.0, 8, 3.0),
-    (3, 1, 8, 130, 16, 4.0, 2, 4.0), (24, 3, 128, 128, 100, 15.0, 64, 4.0)])
+    (3, 1, 8, 130, 16, 4.0, 2, 4.0), (24, 3, 128, 128, 100, 15.0, 64, 4.0), (4, 2, 256, 256, 50, 9.0, 128, 2.0)])
 def test_chunked_attention_alone(heads, kv, dim, vdim, chunk, cap, rot, factor, dtype):
     """biases, norms per head, rotation with scaled frequencies, capped scores, chunks that end inside pages, tiles and
     portions, the output gate"""
