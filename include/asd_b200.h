@@ -641,8 +641,8 @@ ASD_API int asd_dikopel_device_error(asd_dikopel_engine_t* e);
  * turn yarn_fast and yarn_slow times over yarn_original positions by a linear ramp to 1 / factor) and multiplies cos and sin by
  * 0.1 ln(factor) + 1.
  * ff_kind 0: none; 1: W_down (gelu_tanh(W_gate h) * W_up h); 2: `experts` layers of size expert_ff of which every token takes
- * the `top` with the largest sigmoid(router logit), each on its input times that score: g = min(W_gate h, limit),
- * u = clamp(W_up h, +-limit), W_down (g sigmoid(1.702 g) (u + 1)), summed.
+ * the `top` with the largest s = sigmoid(router logit); an expert reads e = s h: a = min(W_gate e, limit), b = W_up e cut to
+ * [-limit, limit], and gives W_down (a sigmoid(1.702 a) (1 + b)); the results are summed.
  *
  * dtype as for the Rivetar engine.  Paged pool: per layer of type 0 or 2 without kv_from [num_pages][page_size][kv_heads *
  * (dim + vdim)], keys then values, layers back to back.  State (caller allocated, fp32), per layer: carried inputs of the
